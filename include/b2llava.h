@@ -228,7 +228,9 @@ int b2_batch_set_row(b2_model* m, b2_kv* kv, int slot, int active, const b2_samp
  * conv is a causal depthwise convolution over time of input_conv_taps taps (0: none; 1: a factor per channel) whose last taps - 1 inputs are carried
  * per slot, for the mixer and for the feed-forward of every layer; B2_BLOCK_PARALLEL_RMS has ONE weighted RMS norm per layer
  * that both sublayers read: x += residual_mult * (mixer(u) + ff(u)), u = rms_w(x).
- * Feed-forwards: B2_FF_CLAMP_GLU (W_down (a(g) (u + 1)) with g = min(W_gate x, ff_limit), u = clamp(W_up x, +-ff_limit),
+ * B2_BLOCK_PARALLEL2: parallel with a norm for each sublayer, x += residual_mult * (mixer(N1(x)) + ff(N2(x))), both norms of the same x. norm_kind of
+ * the two parallel blocks: weighted RMS norm, or the dynamic tanh N(x) = tanh(alpha x) w + b (no statistics; alpha one number).
+ * Feed-forwards: B2_FF_GELU (W_down gelu(W_up x), the erf form), B2_FF_CLAMP_GLU (W_down (a(g) (u + 1)) with g = min(W_gate x, ff_limit), u = clamp(W_up x, +-ff_limit),
  * a(g) = g sigmoid(ff_act_slope g)), B2_FF_RELU_SQ (W_down relu(W_up x)^2), B2_FF_POLYNORM (biased projections around
  * a N(z) + b N(z^2) + c N(z^3) + e, N = division by the token's root mean square), B2_FF_MOE (router, group-limited
  * top-k, experts without biases, optional shared expert; moe_score: sigmoid or softmax scores; moe_group_score: a group counts
@@ -236,17 +238,22 @@ int b2_batch_set_row(b2_model* m, b2_kv* kv, int slot, int active, const b2_samp
  * sum and scaled; moe_act: SiLU-gated experts or W_down relu(W_up x)^2).
  * A model may add a hashed bigram row to every token embedding, loop a block of layers several times with the same tensors
  * (every pass has its own cache/state; before a pass the embedding output is added again from the second pass on, and a
- * learned per-pass vector always; loop_plain: nothing is added between the passes), scale its token embedding, and soft-cap its
- * logits with tanh.
+ * learned per-pass vector always; loop_plain: nothing is added between the passes; loop_mix: x becomes W_in [x; embedding output] in front
+ * of every pass), scale its token embedding, use the embedding table as its head, and soft-cap its logits with tanh.
  * The reference has no such models (its LLMs are HF LLaMA / MPT, llava/model/language_model/); what is shared with the
  * LLaVA path is everything around the layers: b2_kv slots and lengths, b2_decode_step / b2_decode_greedy / b2_stream_* /
  * b2_batch_* (CUDA-graph decode step, device-side token selection, host token ring, continuous batching).
  * compute: B2_COMPUTE_BF16 = bf16 x bf16 -> fp32 matrix products on bf16 weights, everything else fp32;
  *          B2_COMPUTE_F32  = true fp32 throughout (weights widened at load, FMA products, no TF32). */
 enum { B2_ARCH_LLAVA = 0, B2_ARCH_LAYER_LIST = 1 };
-enum { B2_MIXER_MAMBA2 = 1, B2_MIXER_PARALLEL = 2, B2_MIXER_LATENT_ATTN = 3, B2_MIXER_HGRN2 = 4, B2_MIXER_GQA_ATTN = 5, B2_MIXER_GLA = 6 };
-enum { B2_FF_RELU_SQ = 0, B2_FF_POLYNORM = 1, B2_FF_MOE = 2, B2_FF_CLAMP_GLU = 3 };
-enum { B2_BLOCK_POST_LN = 0, B2_BLOCK_PRE_RMS1 = 1, B2_BLOCK_SANDWICH_RMS = 2, B2_BLOCK_PARALLEL_RMS = 3 };
+enum { B2_MIXER_MAMBA2 = 1, B2_MIXER_PARALLEL = 2, B2_MIXER_LATENT_ATTN = 3, B2_MIXER_HGRN2 = 4, B2_MIXER_GQA_ATTN = 5, B2_MIXER_GLA = 6, B2_MIXER_MLSTM = 7,
+       B2_MIXER_DELTA = 8 };
+enum { B2_FF_RELU_SQ = 0, B2_FF_POLYNORM = 1, B2_FF_MOE = 2, B2_FF_CLAMP_GLU = 3, B2_FF_GELU = 4 };
+enum { B2_BLOCK_POST_LN = 0, B2_BLOCK_PRE_RMS1 = 1, B2_BLOCK_SANDWICH_RMS = 2, B2_BLOCK_PARALLEL_RMS = 3, B2_BLOCK_PARALLEL2 = 4 };
+enum { B2_NORM_RMS = 0, B2_NORM_DYT = 1 };
+enum { B2_QK_NORM_NONE = 0, B2_QK_NORM_HEAD = 1, B2_QK_NORM_ALL = 2 };
+enum { B2_SINK_NONE = 0, B2_SINK_FIXED = 1, B2_SINK_HEAD = 2 };
+enum { B2_ROT_YARN = 0, B2_ROT_BANDS = 1 };
 enum { B2_GATE_CHANNEL = 0, B2_GATE_HEAD = 1, B2_GATE_NONE = 2 };
 enum { B2_MASK_CAUSAL = 0, B2_MASK_WINDOW = 1, B2_MASK_CHUNK = 2 };
 enum { B2_MOE_SCORE_SIGMOID = 0, B2_MOE_SCORE_SOFTMAX = 1 };
@@ -282,7 +289,7 @@ typedef struct b2_seq_layer_desc {
     int32_t la_kv_from;      /* 1 + the earlier layer whose cache rows this layer reads; 0: its own */
     /* B2_MIXER_GQA_ATTN */
     int32_t ga_heads, ga_kv_heads, ga_dim, ga_vdim, ga_conv;   /* ga_conv: taps of the convolution on q, k, v (0: none) */
-    int32_t ga_rot_values, ga_sink;
+    int32_t ga_rot_values, ga_sink;   /* ga_sink: B2_SINK_* (HEAD: a learned number per head, mix.sink) */
     float ga_scale, ga_sink_value;
     /* visible keys and rotation of the attention mixers above */
     int32_t mask_kind, mask_size;   /* B2_MASK_* */
@@ -291,7 +298,8 @@ typedef struct b2_seq_layer_desc {
     /* B2_MIXER_GQA_ATTN, further forms (zero: one map, no q / k norm, neighbouring pairs, a gate per channel) */
     int32_t ga_maps;         /* 2: differential attention (two maps per head over the same values); 0 or 1: one map */
     float ga_diff;           /* ga_maps == 2: the constant of lambda, and 1 - ga_diff scales the head's output */
-    int32_t ga_qk_norm;      /* weighted RMS norm of every query and key head (weights shared by the heads) before the rotation */
+    int32_t ga_qk_norm;      /* B2_QK_NORM_*: weighted RMS norm before the rotation, of every query and key head (HEAD; weights shared by the heads) or
+                                of the whole query and the whole key projection (ALL; a weight for every entry) */
     int32_t ga_rot_half;     /* rotated pairs are (m, m + rot_dims / 2) */
     int32_t ga_gate;         /* B2_GATE_* */
     int32_t mask_keep;       /* B2_MASK_WINDOW: the first mask_keep positions of a sequence stay visible */
@@ -300,6 +308,14 @@ typedef struct b2_seq_layer_desc {
     float gl_tau;
     /* B2_FF_CLAMP_GLU */
     float ff_limit, ff_act_slope;
+    /* B2_MIXER_GQA_ATTN: the values are the keys as projected (before norm and rotation; ga_vdim == ga_dim, no mix.v) */
+    int32_t ga_key_values;
+    int32_t rot_scaling;     /* B2_ROT_*: how rot_factor > 0 scales the frequencies (BANDS: rot_slow / rot_fast are the low / high band factors) */
+    /* B2_MIXER_MLSTM: matrix memory with exponential gates, capped at ml_cap by tanh */
+    int32_t ml_heads, ml_dim, ml_vdim;
+    float ml_cap;
+    /* B2_MIXER_DELTA: gated delta rule behind a convolution of dn_conv taps with SiLU on q, k, v; dn_kv_heads query / key heads */
+    int32_t dn_heads, dn_kv_heads, dn_dim, dn_vdim, dn_conv;
 } b2_seq_layer_desc;
 typedef struct b2_seq_model_desc {
     int32_t width, vocab, n_layers;
@@ -317,6 +333,9 @@ typedef struct b2_seq_model_desc {
     int32_t input_conv_taps; /* B2_BLOCK_SANDWICH_RMS: taps of the convolution every sublayer's input passes (0: none) */
     float embed_scale;       /* factor on the token embedding; 0 = 1 */
     int32_t loop_plain;      /* the passes of the looped block follow one another with nothing added in between (no loop.step tensor) */
+    int32_t norm_kind;       /* B2_NORM_*, of B2_BLOCK_PARALLEL_RMS / PARALLEL2 */
+    int32_t tied_head;       /* logits = embed N(x): no head tensor */
+    int32_t loop_mix;        /* parallel blocks: x <- W_in [x; x0] in front of every pass, x0 the embedding output (tensor loop.in; no loop.step) */
 } b2_seq_model_desc;
 int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* layers, b2_model** out);
 /* Layer RUNS of one forward pass (a looped layer counts every time): rows of b2_append_tokens' resid_out; -1 for other models */
@@ -332,7 +351,10 @@ int b2_seq_model_runs(const b2_model* m);
  * l<i>.mix.{q,k,v,q.conv,k.conv,v.conv,g,o} (grouped attention), l<i>.mlp.{router,e<j>.up,e<j>.down,shared.up,shared.down}.
  * B2_BLOCK_PARALLEL_RMS models: embed, head, final.norm, l<i>.norm1 (width each), l<i>.mix.{q,k,v,o} with, by the layer's options,
  * {q,k,v}.conv, {q,k}.norm, g, {lq1,lk1,lq2,lk2} (grouped attention), l<i>.mix.{q,k,v,g,a1,a2,a2.b,norm,o} (gated linear attention),
- * l<i>.mlp.{gate,up,down}. */
+ * l<i>.mlp.{gate,up,down}.
+ * B2_BLOCK_PARALLEL2 models: the same with l<i>.norm2; with norm_kind DYT every norm also has .b (width) and .alpha (one number); tied_head: no
+ * head; loop_mix: loop.in [width, 2 width] (x's columns first); l<i>.mix.{q,k,v,g,i,i.b,f,f.b,norm,o} (mLSTM),
+ * l<i>.mix.{q,k,v,q.conv,k.conv,v.conv,b,a,A_log,dt_bias,g,norm,o} (delta rule), mix.sink (grouped attention with B2_SINK_HEAD). */
 /* Feed the next n tokens of the request in cache slot `slot` (a portion of its prompt, or all of it): the slot's state and
  * key/value rows continue from its current length, or from an empty sequence when restart != 0 (whatever the slot held
  * is then dead: nothing needs clearing). want_host lists n_want indices into these n tokens whose logits are written to

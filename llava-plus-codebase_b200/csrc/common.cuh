@@ -69,6 +69,7 @@ __device__ __forceinline__ float epi_post_act(float v, int post) {
         case 2: return 1.f / (1.f + expf(-v));      // sigmoid
         case 3: return tanhf(v);
         case 4: { const float r = v > 0.f ? v : 0.f; return r * r; }  // relu^2
+        case 5: return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));  // GELU, erf form
         default: return v;
     }
 }

@@ -272,7 +272,9 @@ int rowmap_decode(const RowMap& rm, const int32_t* len, const SampleState* sstat
                   cudaStream_t stream);
 
 // ---- generic Linear on fp32 activations (linear_generic.cu): any M, N, K -----------------------------------------------
-enum { LIN_NONE = 0, LIN_SILU = 1, LIN_SIGMOID = 2, LIN_TANH = 3, LIN_RELU_SQ = 4 };
+enum { LIN_NONE = 0, LIN_SILU = 1, LIN_SIGMOID = 2, LIN_TANH = 3, LIN_RELU_SQ = 4, LIN_GELU = 5 };   // LIN_GELU: the exact (erf) form
+// Dynamic-tanh norm, element by element and without statistics: N(x)[c] = tanh(alpha[0] x[c]) w[c] + b[c] (device pointers)
+struct DytNorm { const float *alpha = nullptr, *w = nullptr, *b = nullptr; };
 struct LinearArgs {
     const float* A = nullptr; int64_t lda = 0;   // fp32 [M, K]
     const void* W = nullptr; int64_t ldw = 0;    // [N, K], DT_BF16 or DT_F32
@@ -284,7 +286,10 @@ struct LinearArgs {
     float alpha = 1.f;                           // out = alpha * act(A W^T + bias) (+ out when accumulate)
     int accumulate = 0;
     int round_a = 0;                             // round A to bf16 first (bf16 compute: the product is bf16 x bf16 -> fp32)
+    DytNorm norm;                                // norm.alpha non-null: A passes this norm while it is staged (linear_fuses_norm calls only)
 };
+// whether a call of these sizes can norm A on its way in: a handful of rows with K % 8 == 0 (the weight-streaming kernel)
+bool linear_fuses_norm(int M, int K);
 int linear_f32(const LinearArgs& a, cudaStream_t stream);
 // out[r, :K] = bf16(A[r, :K]): the A operand of a tensor-core GEMM from fp32 activations (ld_out % 8 == 0)
 int cast_rows_bf16(const float* A, int64_t lda, void* out, int64_t ld_out, int M, int K, cudaStream_t stream);
@@ -359,9 +364,12 @@ int layernorm_gather_f32(const float* x, const int32_t* row_index, const float* 
 // Per row and per group of `group` consecutive channels (cols % group == 0):
 //   gate_first: out = unit_rms(y * silu(z)) * gamma            (state-space mixer: the gate comes before the norm)
 //   otherwise : out = unit_rms(y) * gamma * silu(z)            (RWKV mixer: per-head norm, then weight, then gate)
-// gamma_shared: one weight vector [group] for every group instead of [cols]
+// gamma_shared: one weight vector [group] for every group instead of [cols]. sigmoid_gate: sigmoid(z) in place of silu(z). den
+// (nullable, [rows, cols / group]): y is divided by it before the norm. out16 (nullable, bf16 [rows, ld_out16]): the result goes there
+// instead of out (the operand of a tensor-core product).
 int gated_group_rmsnorm_f32(const float* y, int64_t ldy, const float* z, int64_t ldz, const float* gamma, float* out, int64_t ldo, int rows,
-                            int cols, int group, int gate_first, float eps, cudaStream_t stream, int gamma_shared = 0);
+                            int cols, int group, int gate_first, float eps, cudaStream_t stream, int gamma_shared = 0, int sigmoid_gate = 0,
+                            const float* den = nullptr, void* out16 = nullptr, int64_t ld_out16 = 0);
 // ungated form; gamma_shared: one weight vector [group] for every group instead of [cols]
 int group_rmsnorm_f32(const float* y, int64_t ldy, const float* gamma, int gamma_shared, float* out, int64_t ldo, int rows, int cols, int group,
                       float eps, cudaStream_t stream);
@@ -402,6 +410,13 @@ int sigmoid_gate_f32(const float* a, int64_t lda, const float* g, int64_t ldg, f
 int rms_weight_f32(const float* in, int64_t ld_in, const int32_t* row_index, const float* w, float* out, int64_t ld_out, int accumulate, int rows,
                    int cols, float eps, cudaStream_t stream);
 
+// One or two dynamic-tanh norms of the same (gathered) rows in one pass: row r of an output is N(x[row_index[r]]) (row_index null: row r),
+// as fp32 (out, pitch cols) or as the bf16 operand of a tensor-core product (out16, pitch cols).
+struct DytOut { DytNorm norm; float* out = nullptr; void* out16 = nullptr; };
+int dyt_rows_f32(const float* x, const int32_t* row_index, const DytOut* outs, int n_outs, int rows, int cols, cudaStream_t stream);
+// out[r] = [a[r] | b[r]], rows of `cols` entries each, as fp32 (out) or bf16 (out16)
+int concat_rows_f32(const float* a, const float* b, float* out, void* out16, int rows, int cols, cudaStream_t stream);
+
 // The norms around a sublayer of a sandwich block in one pass over a row: first (y, w_post non-null) x += rms_w_post(y), the normed
 // output of the previous sublayer joining the residual stream; then (w_pre non-null) out = rms_w_pre(x), the next sublayer's input.
 // With conv_w the input convolution of a decode step rides along: every row is a segment of ONE token (row r = segs[r]), conv_out =
@@ -417,10 +432,14 @@ struct SandwichNormArgs {
 int sandwich_norm_f32(const SandwichNormArgs& a, cudaStream_t stream);
 
 // ---- rotary positions (rotary.cu) -------------------------------------------------------------------------------------------
-// Pairs (2m, 2m+1) (or, in the half layout, (m, m + pairs)), m < floor(dims / 2), turn by position * f_m, f_m = base^(-2m / dims). factor > 0: f_m is blended towards f_m / factor
+// Pairs (2m, 2m+1) (or, in the half layout, (m, m + pairs)), m < floor(dims / 2), turn by position * f_m, f_m = base^(-2m / dims). factor > 0, scaling
+// ROT_YARN: f_m is blended towards f_m / factor
 // over the pairs between lo = max(floor(dim(fast)), 0) and hi = min(ceil(dim(slow)), dims - 1), dim(t) = dims ln(original / (2 pi t)) /
 // (2 ln base), and cos / sin are scaled by 0.1 ln(factor) + 1.
-struct RotaryDesc { int dims = 0; float base = 10000.f, factor = 0.f, original = 0.f, fast = 0.f, slow = 0.f; };
+// factor > 0, scaling ROT_BANDS: f_m stays where its wavelength l = 2 pi / f_m is below original / fast, becomes f_m / factor above original / slow,
+// and (1 - s) f_m / factor + s f_m, s = (original / l - slow) / (fast - slow), in between; cos / sin are not scaled.
+enum { ROT_YARN = 0, ROT_BANDS = 1 };   // the values of B2_ROT_*
+struct RotaryDesc { int dims = 0; float base = 10000.f, factor = 0.f, original = 0.f, fast = 0.f, slow = 0.f; int scaling = ROT_YARN; };
 // table_dev[p][m] = (cos, sin)(p * f_m) * scale for p < positions; computed on the host in double precision
 int rotary_table_build(const RotaryDesc& d, int positions, float2* table_dev);
 // For every live row r (position row_pos[r] >= 0) and head h < heads: the head's `size` entries at in[r * ld_in + h * hs_in] are copied
@@ -438,6 +457,8 @@ struct RotateArgs {
     int half = 0;                                // pair m is (offset + m, offset + m + pairs) instead of (offset + 2m, offset + 2m + 1)
     const float* norm_w = nullptr; float eps = 0.f;   // non-null: the head is first normed, x / sqrt(mean(x^2) + eps) * norm_w over its `size` entries
                                                       // (one weight vector for all heads); such calls run one warp per (row, head)
+    int norm_all = 0;                            // the norm runs over all heads * size entries together, with a weight for each (norm_w[heads * size]); such
+                                                 // calls run one CTA per row and part (heads adjoining in the input: hs_in == size)
 };
 int rotate_rows_f32(const RotateArgs& a, cudaStream_t stream);
 // up to three such calls over the same rows in one launch (queries, keys and values of an attention layer)
@@ -486,6 +507,32 @@ struct ScanArgs {
     const SeqSeg* segs = nullptr; int nseg = 0;
 };
 int linear_scan_f32(const ScanArgs& a, cudaStream_t stream);
+
+// ---- matrix memories with one decay per head (matrix_memory.cu) ------------------------------------------------------------------
+// A [key, value] state per head, written once per token and read in the same token:
+//   MEM_DELTA: gated delta rule. k^ = k / sqrt(sum k^2 + 1e-6), q^ likewise times q_scale; beta = sigmoid(gate1); g = exp(-exp(a_log[h])
+//              softplus(gate2 + bias2[h])); S <- g S; S <- S + k^ (beta (v - S^T k^))^T; y = S^T q^. kv_heads q / k heads serve heads / kv_heads
+//              consecutive value heads each.
+//   MEM_MLSTM: exponential gates under a running maximum m (0 at a sequence start). i = cap tanh((gate1 + bias1[h]) / cap),
+//              f = log_sigmoid(cap tanh((gate2 + bias2[h]) / cap)); m' = max(f + m, i); S <- exp(f + m - m') S + exp(i - m') k v^T, n likewise with
+//              k alone; y = S^T (q_scale q), den = max(|n . (q_scale q)|, exp(-m')) + 1e-6 (the caller divides y by it).
+// The state is [slots][heads][columns][dk] fp32, columns = dv (MEM_MLSTM: dv + 1, n is the last one); mem_blocks(columns) column blocks of a
+// head carry one m each: run_max [slots][heads][mem_blocks].
+enum { MEM_DELTA = 0, MEM_MLSTM = 1 };
+struct MemoryArgs {
+    int mode = MEM_DELTA;
+    const float *q = nullptr, *k = nullptr, *v = nullptr; int64_t ldq = 0, ldk = 0, ldv = 0;   // [rows, kv_heads * dk] x 2, [rows, heads * dv]
+    const float *gate1 = nullptr, *gate2 = nullptr; int64_t ldg = 0;                            // [rows, heads] raw projections
+    const float *bias1 = nullptr, *bias2 = nullptr, *a_log = nullptr;                           // [heads]
+    float q_scale = 1.f, cap = 1.f;
+    float *state = nullptr, *run_max = nullptr;
+    float* y = nullptr; int64_t ldy = 0;                                                         // [rows, heads * dv]
+    float* den = nullptr;                                                                        // MEM_MLSTM: [rows, heads]
+    int heads = 0, kv_heads = 0, dk = 0, dv = 0;                                                  // dk <= 256
+    const SeqSeg* segs = nullptr; int nseg = 0;
+};
+int mem_blocks(int columns);
+int matrix_memory_f32(const MemoryArgs& a, cudaStream_t stream);
 
 // ---- attention with unit-RMS q/k, query temperature, tanh soft-cap and a bucketed distance bias (attention_bias.cu) -----
 enum { MASK_CAUSAL = 0, MASK_WINDOW = 1, MASK_CHUNK = 2 };

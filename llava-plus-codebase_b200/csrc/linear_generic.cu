@@ -20,6 +20,7 @@ __device__ __forceinline__ float lin_act(float v, int act) {
         case LIN_SIGMOID: return 1.f / (1.f + expf(-v));
         case LIN_TANH: return tanhf(v);
         case LIN_RELU_SQ: { const float r = v > 0.f ? v : 0.f; return r * r; }
+        case LIN_GELU: return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
         default: return v;
     }
 }
@@ -50,7 +51,7 @@ constexpr int RW_COLS = 2, RW_SMEM_FLOATS = 16384;
 template <typename TW>
 __global__ void __launch_bounds__(256) linear_rows_vec_kernel(const float* __restrict__ A, int64_t lda, const TW* __restrict__ W, int64_t ldw,
                                                               const float* __restrict__ bias, float* __restrict__ out, int64_t ld_out, int M, int N,
-                                                              int K, int kc_max, int act, float alpha, int accumulate, int round_a) {
+                                                              int K, int kc_max, int act, float alpha, int accumulate, int round_a, DytNorm norm) {
     extern __shared__ float sA[];  // [M][kc]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int ngroups = (N + 8 * RW_COLS - 1) / (8 * RW_COLS);
@@ -61,6 +62,12 @@ __global__ void __launch_bounds__(256) linear_rows_vec_kernel(const float* __res
         for (int e = threadIdx.x * 4; e < M * kc; e += 1024) {
             const int m = e / kc, k = e % kc;
             float4 v = *reinterpret_cast<const float4*>(A + (size_t)m * lda + kc0 + k);
+            if (norm.alpha != nullptr) {   // a norm without statistics is applied on the way in: no pass of its own over A
+                const float al = norm.alpha[0];
+                const float4 w = *reinterpret_cast<const float4*>(norm.w + kc0 + k), b = *reinterpret_cast<const float4*>(norm.b + kc0 + k);
+                v.x = fmaf(tanhf(al * v.x), w.x, b.x); v.y = fmaf(tanhf(al * v.y), w.y, b.y);
+                v.z = fmaf(tanhf(al * v.z), w.z, b.z); v.w = fmaf(tanhf(al * v.w), w.w, b.w);
+            }
             if (round_a) { v.x = round_bf16(v.x); v.y = round_bf16(v.y); v.z = round_bf16(v.z); v.w = round_bf16(v.w); }
             *reinterpret_cast<float4*>(sA + e) = v;
         }
@@ -225,16 +232,18 @@ int launch_linear(const LinearArgs& a, cudaStream_t st) {
                 const int grid = a.K <= kc_max ? std::min(ngroups, 3 * num_sms()) : ngroups;
                 const size_t smem = (size_t)a.M * std::min(kc_max, a.K) * sizeof(float);
                 linear_rows_vec_kernel<TW><<<grid, 256, smem, st>>>(a.A, a.lda, W, a.ldw, a.bias, a.out, a.ld_out, a.M, a.N, a.K, kc_max, a.act,
-                                                                  a.alpha, a.accumulate, a.round_a);
+                                                                  a.alpha, a.accumulate, a.round_a, a.norm);
                 B2_LAUNCH_CHECK();
                 return 0;
             }
         }
         {
+            B2_CHECK_ARG(a.norm.alpha == nullptr, "linear: a norm on the way in needs the vectorised row kernel (K=%d, lda=%lld)", a.K, (long long)a.lda);
             linear_rows_kernel<TW><<<(a.N + 7) / 8, 256, 0, st>>>(a.A, a.lda, W, a.ldw, a.bias, a.out, a.ld_out, a.M, a.N, a.K, a.act, a.alpha,
                                                                  a.accumulate, a.round_a);
         }
     } else {
+        B2_CHECK_ARG(a.norm.alpha == nullptr, "linear: a norm on the way in is for at most %d rows (got %d)", MR, a.M);
         dim3 grid((a.N + TB - 1) / TB, (a.M + TB - 1) / TB);
         linear_tiled_kernel<TW><<<grid, 256, 0, st>>>(a.A, a.lda, W, a.ldw, a.bias, a.out, a.ld_out, a.M, a.N, a.K, a.act, a.alpha,
                                                       a.accumulate, a.round_a);
@@ -460,6 +469,10 @@ int cast_rows_bf16(const float* A, int64_t lda, void* out, int64_t ld_out, int M
     B2_LAUNCH_CHECK();
     return 0;
 }
+
+// The row kernel takes K in chunks when the rows do not fit its staging buffer whole; an activation then rules it out, so the fused norm
+// is offered only where K fits.
+bool linear_fuses_norm(int M, int K) { return M >= 1 && M <= MR && K % 8 == 0 && K <= RW_SMEM_FLOATS / M / 8 * 8; }
 
 int linear_f32(const LinearArgs& a, cudaStream_t st) {
     B2_CHECK_ARG(a.A && a.W && a.out && a.M > 0 && a.N > 0 && a.K > 0, "linear: bad argument (M=%d N=%d K=%d)", a.M, a.N, a.K);

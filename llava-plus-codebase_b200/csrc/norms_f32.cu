@@ -1,7 +1,8 @@
 // fp32 normalisations and row helpers of the layer-list decoders: LayerNorm of a sublayer's output added to the residual
 // stream, gathered LayerNorm in front of the output head, grouped unit-RMS norm with a SiLU gate (before or after the
 // norm), embedding rows as fp32, the row map of a call; for pre-norm blocks: the one-number RMS norm (with the opening of a
-// looped pass folded in), the weighted RMS norm (plain, gathered, or added onto the residual stream), PolyNorm, the logit soft-cap, per-head sigmoid gates, token + hashed-bigram embedding, and the
+// looped pass folded in), the weighted RMS norm (plain, gathered, or added onto the residual stream), PolyNorm, the dynamic-tanh norm
+// (element by element, up to two norms of a row in one pass), the logit soft-cap, per-head sigmoid gates, token + hashed-bigram embedding, and the
 // normalised latent row of a low-rank key/value cache. Statistics, sums and outputs are fp32 throughout; any width.
 #include "common.cuh"
 #include "kernels.h"
@@ -66,25 +67,77 @@ __device__ __forceinline__ float silu_f(float v) { return v / (1.f + expf(-v)); 
 // one warp per (row, group)
 __global__ void gated_group_rmsnorm_kernel(const float* __restrict__ y, int64_t ldy, const float* __restrict__ z, int64_t ldz,
                                            const float* __restrict__ gamma, float* __restrict__ out, int64_t ldo, int rows, int groups, int group,
-                                           int gate_first, int gamma_shared, float eps) {
+                                           int gate_first, int gamma_shared, float eps, int sigmoid_gate, const float* __restrict__ den,
+                                           __nv_bfloat16* __restrict__ out16, int64_t ldo16) {
     const int w = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (w >= rows * groups) return;
     const int r = w / groups, g = w % groups;
     const float* yr = y + (size_t)r * ldy + (size_t)g * group;
     const float* zr = z != nullptr ? z + (size_t)r * ldz + (size_t)g * group : nullptr;   // null: no gate
     const float* gm = gamma + (gamma_shared ? 0 : (size_t)g * group);                      // one weight vector for all groups, or one each
+    const float pre = den != nullptr ? 1.f / den[(size_t)r * groups + g] : 1.f;
     float q = 0.f;
     for (int c = lane; c < group; c += 32) {
-        const float v = (gate_first && zr != nullptr) ? yr[c] * silu_f(zr[c]) : yr[c];
+        const float v = ((gate_first && zr != nullptr) ? yr[c] * silu_f(zr[c]) : yr[c]) * pre;
         q = fmaf(v, v, q);
     }
     q = warp_sum(q);
-    const float rinv = 1.f / sqrtf(q / (float)group + eps);
+    const float rinv = pre / sqrtf(q / (float)group + eps);
     float* o = out + (size_t)r * ldo + (size_t)g * group;
+    __nv_bfloat16* o16 = out16 != nullptr ? out16 + (size_t)r * ldo16 + (size_t)g * group : nullptr;
     for (int c = lane; c < group; c += 32) {
-        const float gz = zr != nullptr ? silu_f(zr[c]) : 1.f;
-        o[c] = gate_first ? (yr[c] * gz) * rinv * gm[c] : yr[c] * rinv * gm[c] * gz;
+        const float gz = zr == nullptr ? 1.f : (sigmoid_gate ? 1.f / (1.f + expf(-zr[c])) : silu_f(zr[c]));
+        const float v = gate_first ? (yr[c] * gz) * rinv * gm[c] : yr[c] * rinv * gm[c] * gz;
+        if (o16 != nullptr) o16[c] = __float2bfloat16_rn(v);
+        else o[c] = v;
     }
+}
+
+// one or two dynamic-tanh norms of a row: the row is read once, 16 bytes at a time where the width allows
+struct DytOuts { DytOut o[2]; };
+__device__ __forceinline__ float dyt_f(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+template <bool VEC>
+__global__ void __launch_bounds__(256) dyt_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ row_index, DytOuts outs, int n_outs,
+                                                       int cols) {
+    const size_t r = blockIdx.y;
+    const float* xr = x + (size_t)(row_index != nullptr ? row_index[r] : (int)r) * cols;
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * (VEC ? 4 : 1);
+    if (c >= cols) return;
+    if (VEC) {
+        const float4 v = *reinterpret_cast<const float4*>(xr + c);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            if (i >= n_outs) break;
+            const DytOut& o = outs.o[i];
+            const float al = o.norm.alpha[0];
+            const float4 w = *reinterpret_cast<const float4*>(o.norm.w + c), b = *reinterpret_cast<const float4*>(o.norm.b + c);
+            const float4 y = make_float4(dyt_f(v.x, al, w.x, b.x), dyt_f(v.y, al, w.y, b.y), dyt_f(v.z, al, w.z, b.z), dyt_f(v.w, al, w.w, b.w));
+            if (o.out16 != nullptr) {
+                __nv_bfloat162* d = reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(o.out16) + r * cols + c);
+                d[0] = __floats2bfloat162_rn(y.x, y.y);
+                d[1] = __floats2bfloat162_rn(y.z, y.w);
+            }
+            if (o.out != nullptr) *reinterpret_cast<float4*>(o.out + r * cols + c) = y;
+        }
+    } else {
+        const float v = xr[c];
+        for (int i = 0; i < n_outs; ++i) {
+            const DytOut& o = outs.o[i];
+            const float y = dyt_f(v, o.norm.alpha[0], o.norm.w[c], o.norm.b[c]);
+            if (o.out16 != nullptr) reinterpret_cast<__nv_bfloat16*>(o.out16)[r * cols + c] = __float2bfloat16_rn(y);
+            if (o.out != nullptr) o.out[r * cols + c] = y;
+        }
+    }
+}
+
+__global__ void __launch_bounds__(256) concat_rows_kernel(const float* __restrict__ a, const float* __restrict__ b, float* __restrict__ out,
+                                                          __nv_bfloat16* __restrict__ out16, int cols) {
+    const size_t r = blockIdx.y;
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= 2 * cols) return;
+    const float v = c < cols ? a[r * cols + c] : b[r * cols + c - cols];
+    if (out16 != nullptr) out16[r * 2 * cols + c] = __float2bfloat16_rn(v);
+    else out[r * 2 * cols + c] = v;
 }
 
 // differential attention: one warp per (row, head) subtracts lambda times the second map's output from the first map's and brings
@@ -451,11 +504,13 @@ int layernorm_gather_f32(const float* x, const int32_t* row_index, const float* 
 }
 
 int gated_group_rmsnorm_f32(const float* y, int64_t ldy, const float* z, int64_t ldz, const float* gamma, float* out, int64_t ldo, int rows,
-                            int cols, int group, int gate_first, float eps, cudaStream_t st, int gamma_shared) {
-    B2_CHECK_ARG(y && z && gamma && out && rows > 0 && group > 0 && cols % group == 0, "gated_group_rmsnorm: cols %d is not a multiple of the group %d",
+                            int cols, int group, int gate_first, float eps, cudaStream_t st, int gamma_shared, int sigmoid_gate, const float* den,
+                            void* out16, int64_t ld_out16) {
+    B2_CHECK_ARG(y && z && gamma && (out || out16) && rows > 0 && group > 0 && cols % group == 0, "gated_group_rmsnorm: cols %d is not a multiple of the group %d",
                  cols, group);
     const int groups = cols / group, warps = rows * groups;
-    gated_group_rmsnorm_kernel<<<(warps + 7) / 8, 256, 0, st>>>(y, ldy, z, ldz, gamma, out, ldo, rows, groups, group, gate_first, gamma_shared, eps);
+    gated_group_rmsnorm_kernel<<<(warps + 7) / 8, 256, 0, st>>>(y, ldy, z, ldz, gamma, out, ldo, rows, groups, group, gate_first, gamma_shared, eps,
+                                                               sigmoid_gate, den, reinterpret_cast<__nv_bfloat16*>(out16), ld_out16);
     B2_LAUNCH_CHECK();
     return 0;
 }
@@ -464,7 +519,8 @@ int group_rmsnorm_f32(const float* y, int64_t ldy, const float* gamma, int gamma
                       float eps, cudaStream_t st) {
     B2_CHECK_ARG(y && gamma && out && rows > 0 && group > 0 && cols % group == 0, "group_rmsnorm: cols %d is not a multiple of the group %d", cols, group);
     const int groups = cols / group, warps = rows * groups;
-    gated_group_rmsnorm_kernel<<<(warps + 7) / 8, 256, 0, st>>>(y, ldy, nullptr, 0, gamma, out, ldo, rows, groups, group, 0, gamma_shared, eps);
+    gated_group_rmsnorm_kernel<<<(warps + 7) / 8, 256, 0, st>>>(y, ldy, nullptr, 0, gamma, out, ldo, rows, groups, group, 0, gamma_shared, eps,
+                                                               0, nullptr, nullptr, 0);
     B2_LAUNCH_CHECK();
     return 0;
 }
@@ -508,6 +564,29 @@ int rms_weight_f32(const float* in, int64_t ld_in, const int32_t* row_index, con
                    int cols, float eps, cudaStream_t st) {
     B2_CHECK_ARG(in && w && out && rows > 0 && cols > 0, "rms_weight: bad argument");
     rms_weight_kernel<<<rows, cols >= 1024 ? 256 : 128, 0, st>>>(in, ld_in, row_index, w, out, ld_out, accumulate, cols, eps);
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+int dyt_rows_f32(const float* x, const int32_t* row_index, const DytOut* outs, int n_outs, int rows, int cols, cudaStream_t st) {
+    B2_CHECK_ARG(x && outs && n_outs >= 1 && n_outs <= 2 && rows > 0 && cols > 0, "dyt_rows: bad argument");
+    DytOuts o;
+    uintptr_t align = reinterpret_cast<uintptr_t>(x);
+    for (int i = 0; i < n_outs; ++i) {
+        o.o[i] = outs[i];
+        const DytNorm& n = outs[i].norm;
+        B2_CHECK_ARG(n.alpha && n.w && n.b && (outs[i].out || outs[i].out16), "dyt_rows: norm %d lacks a tensor or an output", i);
+        align |= reinterpret_cast<uintptr_t>(n.w) | reinterpret_cast<uintptr_t>(n.b) | reinterpret_cast<uintptr_t>(outs[i].out) | reinterpret_cast<uintptr_t>(outs[i].out16);
+    }
+    if (cols % 4 == 0 && (align & 15) == 0) dyt_rows_kernel<true><<<dim3((cols / 4 + 255) / 256, rows), 256, 0, st>>>(x, row_index, o, n_outs, cols);
+    else dyt_rows_kernel<false><<<dim3((cols + 255) / 256, rows), 256, 0, st>>>(x, row_index, o, n_outs, cols);
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
+int concat_rows_f32(const float* a, const float* b, float* out, void* out16, int rows, int cols, cudaStream_t st) {
+    B2_CHECK_ARG(a && b && (out || out16) && rows > 0 && cols > 0, "concat_rows: bad argument");
+    concat_rows_kernel<<<dim3((2 * cols + 255) / 256, rows), 256, 0, st>>>(a, b, out, reinterpret_cast<__nv_bfloat16*>(out16), cols);
     B2_LAUNCH_CHECK();
     return 0;
 }

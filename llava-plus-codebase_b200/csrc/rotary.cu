@@ -2,11 +2,11 @@
 // (m, m + pairs)) turn by position * f_m.
 // cos and sin come from a table [position][pair] that the cache builds on the host in double precision (the plain
 // frequencies base^(-2m/dims), optionally blended towards f_m / factor over a ramp of pairs with cos / sin scaled, the long-context
-// form known as YaRN), so an angle never carries the rounding of a 32-bit product of a large position. One kernel serves
+// form known as YaRN, or scaled by bands of wavelength), so an angle never carries the rounding of a 32-bit product of a large position. One kernel serves
 // queries (in place), keys and values on their way into the cache slabs, a rotated part copied to another layout, and the
 // turn back of an attention output by its query's position with the sigmoid output gate applied in the same pass. When a head is
 // normed before it turns (weighted RMS norm over the head, one weight vector for all heads), one warp takes a (row, head): it sums
-// the squares, then every lane norms and turns the pairs it owns. A further kernel writes the row of a low-rank key/value cache that
+// the squares, then every lane norms and turns the pairs it owns. A norm over all heads of a projection together takes a CTA per row and part. A further kernel writes the row of a low-rank key/value cache that
 // holds a normed latent AND one rotated key part.
 #include <math.h>
 
@@ -104,6 +104,48 @@ __global__ void __launch_bounds__(256) rotate_rows_warp_kernel(RotateParts ps, i
     }
 }
 
+// One CTA per (row, part): the optional norm runs over ALL heads of the part together (a weight for each of its heads * size entries),
+// then every head's pairs turn. Parts may read the same input (values that are the raw keys), so a part writes in place only what no
+// other part reads.
+__global__ void __launch_bounds__(256) rotate_rows_block_kernel(RotateParts ps) {
+    __shared__ float red[8];
+    const RotateArgs& a = ps.p[blockIdx.y];
+    const int r = blockIdx.x, tid = threadIdx.x;
+    const int pos = a.row_pos[r];
+    if (pos < 0) return;
+    const float* src = a.in + (size_t)r * a.ld_in;
+    float mul = 1.f;
+    if (a.norm_w != nullptr) {
+        const int n = a.heads * a.size;
+        float q = 0.f;
+        for (int d = tid; d < n; d += 256) q = fmaf(src[d], src[d], q);
+        q = warp_sum(q);
+        if ((tid & 31) == 0) red[tid >> 5] = q;
+        __syncthreads();   // also: every entry has been read before any is written in place (each thread then re-reads only what it writes)
+        q = ((red[0] + red[1]) + (red[2] + red[3])) + ((red[4] + red[5]) + (red[6] + red[7]));
+        mul = 1.f / sqrtf(q / (float)n + a.eps);
+    }
+    const int units = a.size - a.pairs;
+    for (int i = tid; i < a.heads * units; i += 256) {
+        const int h = i / units, u = i - h * units;
+        const float* s = src + (size_t)h * a.hs_in;
+        float* dst = a.cache != nullptr ? a.cache + (((size_t)a.row_slot[r] * a.heads + h) * a.Smax + pos) * a.size
+                                        : a.out + (size_t)r * a.ld_out + (size_t)h * a.hs_out;
+        const float* nw = a.norm_w != nullptr ? a.norm_w + (size_t)h * a.size : nullptr;
+        if (u >= a.offset && u < a.offset + a.pairs) {
+            const int mp = u - a.offset, d = a.half ? a.offset + mp : a.offset + 2 * mp, d2 = a.half ? d + a.pairs : d + 1;
+            const float2 cs = a.table[(size_t)pos * a.pairs + mp];
+            float x = s[d], y = s[d2];
+            if (nw != nullptr) { x = x * mul * nw[d]; y = y * mul * nw[d2]; }
+            dst[d] = x * cs.x - y * cs.y;
+            dst[d2] = y * cs.x + x * cs.y;
+        } else {
+            const int d = u < a.offset ? u : u + a.pairs;
+            dst[d] = nw != nullptr ? s[d] * mul * nw[d] : s[d];
+        }
+    }
+}
+
 // cache[slot][pos] = [ unit_rms(in[r, :rank]) * gamma | the rot entries behind them, their first `pairs` pairs turned by pos ]
 __global__ void __launch_bounds__(128) latent_rot_append_kernel(const float* __restrict__ in, int64_t ld_in, const float* __restrict__ gamma,
                                                                 float* __restrict__ cache, const int32_t* __restrict__ row_slot,
@@ -147,7 +189,7 @@ int rotate_rows_multi_f32(const RotateArgs* parts, int n, cudaStream_t st) {
     B2_CHECK_ARG(parts && n >= 1 && n <= 3, "rotate_rows_multi: 1..3 parts");
     RotateParts ps;
     int units = 0, heads = 0;
-    bool normed = false;
+    bool normed = false, whole = false;
     for (int i = 0; i < n; ++i) {
         const RotateArgs& a = parts[i];
         B2_CHECK_ARG(a.in && (a.out || a.cache) && (a.table || a.pairs == 0) && a.row_pos && a.rows == parts[0].rows && a.heads > 0 && a.size > 0, "rotate_rows_multi: bad argument");
@@ -156,7 +198,15 @@ int rotate_rows_multi_f32(const RotateArgs* parts, int n, cudaStream_t st) {
         ps.p[i] = a;
         units = std::max(units, a.heads * (a.size - a.pairs));
         normed = normed || a.norm_w != nullptr;
+        whole = whole || a.norm_all;
+        B2_CHECK_ARG(!a.norm_all || (a.norm_w && a.hs_in == a.size && !a.inverse && a.gate == nullptr), "rotate_rows_multi: a norm over all heads takes adjoining heads, no gate");
         heads += a.heads;
+    }
+    if (whole) {   // one CTA per row and part
+        for (int i = 0; i < n; ++i) B2_CHECK_ARG(parts[i].norm_w == nullptr || parts[i].norm_all, "rotate_rows_multi: norms per head and over all heads do not mix");
+        rotate_rows_block_kernel<<<dim3(parts[0].rows, n), 256, 0, st>>>(ps);
+        B2_LAUNCH_CHECK();
+        return 0;
     }
     if (normed) {   // a normed head needs its sum of squares: one warp per (row, head) of every part
         rotate_rows_warp_kernel<<<dim3((heads + 7) / 8, parts[0].rows), 256, 0, st>>>(ps, n);
@@ -183,6 +233,15 @@ void rotary_frequencies(const RotaryDesc& d, std::vector<double>& freq, double& 
     for (int i = 0; i < pairs; ++i) freq[i] = pow((double)d.base, -2.0 * i / d.dims);
     if (!(d.factor > 0.f)) return;
     const double two_pi = 6.283185307179586476925286766559;
+    if (d.scaling == ROT_BANDS) {
+        for (int i = 0; i < pairs; ++i) {
+            const double turns = d.original * freq[i] / two_pi;   // original / wavelength
+            if (turns > d.fast) continue;
+            const double s = turns < d.slow ? 0.0 : (turns - d.slow) / ((double)d.fast - d.slow);
+            freq[i] = (1.0 - s) * freq[i] / d.factor + s * freq[i];
+        }
+        return;
+    }
     auto turn_dim = [&](double turns) { return d.dims * log((double)d.original / (two_pi * turns)) / (2.0 * log((double)d.base)); };
     const double lo = std::max(floor(turn_dim(d.fast)), 0.0), hi = std::min(ceil(turn_dim(d.slow)), (double)d.dims - 1.0);
     for (int i = 0; i < pairs; ++i) {

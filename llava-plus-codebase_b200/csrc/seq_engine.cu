@@ -31,6 +31,9 @@ struct SeqWeights {   // tensors of one layer that owns its weights
     DevBuf qn_w, kn_w, lam4;                            // grouped attention, further forms: weights of the q / k norm; [lq1 | lk1 | lq2 | lk2] of
     float lambda = 0.f;                                 // differential attention and the layer's lambda (made from them when the model is finalized)
     DevBuf gla_w, a2_w, a2_b, gnorm;                    // gated linear attention: [q | k | v | g | a1] fused, W_a2 and its bias, the heads' norm weight
+    DevBuf norm1_a, norm2_a;                            // dynamic tanh: the norms' slopes (one number each; the bias lies in norm1_b / norm2_b)
+    DevBuf mem_w, mnorm_w, gate1_b, gate2_b;            // matrix memories: [q | k | v | two gates | g] fused, norm weight, biases of the gates (mLSTM:
+                                                        // input, forget; the delta rule's decay bias and logarithm lie in dt_bias / a_log)
     std::map<std::string, int> got;
 };
 
@@ -45,9 +48,11 @@ struct SeqLayerInfo {
     int pq = 0, pproj = 0, pproj_ld = 0;              // latent attention / HGRN2: width of q, of the fused projection, its pitch
     int pv = 0;                                       // heads * vdim of those mixers
     int lqw = 0, lqw_ld = 0, lrow = 0;                // latent attention: heads * (dim + rot_dim) and its pitch, a cache row (rank + rot_dim)
+    int pk = 0;                                       // matrix memories: width of q and of k (pv: of v and of the gate)
     int maps = 1, gw = 0;                             // grouped attention: score maps per head (2: differential), width of the gate projection
 };
-struct SeqRun { int layer; int pass; int kv_run; };   // one layer run; pass >= 0: the run opens pass `pass` of the looped block; kv_run: the run
+struct SeqRun { int layer; int pass; int kv_run; };   // one layer run; pass >= 0: the run opens pass `pass` of the looped block and something is added
+                                                      // or mixed in there; kv_run: the run
                                                       // whose cache rows a borrowing latent-attention layer reads (-1: its own)
 
 struct SeqModel {
@@ -55,9 +60,11 @@ struct SeqModel {
     std::vector<SeqLayerInfo> layers;
     std::vector<SeqRun> runs;          // what one forward pass executes, in order (a looped layer appears once per pass)
     std::vector<SeqWeights> w;
-    DevBuf embed, head, final_w, final_b;
+    DevBuf embed, head, final_w, final_b, final_a;
     DevBuf bigram, loop_step;          // [buckets + 1, width] in the weight dtype; [times, width] fp32
     DevBuf x0;                         // the embedding output, kept for the passes of a looped block
+    DevBuf loop_in, cat;               // looped block with an input mix: W_in [width, 2 width], rows [x | x0] in fp32
+    DevBuf h2, h1_16, h2_16, f16, den;        // parallel block with two norms: the feed-forward's input (fp32 / bf16), its activated rows as bf16; mLSTM normalisers
     DevBuf hin;                        // sandwich block: a sublayer's input after its convolution
     DevBuf qabs, olat;                 // latent attention: queries carried into the latent space, latent-space outputs [rows, heads*rank]
     DevBuf ffa;                        // activated feed-forward rows
@@ -79,7 +86,8 @@ struct SeqLayerState {
     DevBuf kc, vc, bucket_of;          // attention: [slots][G][Smax][dk], [slots][G][Smax][dv], int32 [Smax]
     DevBuf wkv, prev;                  // RWKV: [slots][heads][dim][dim], [slots][width]
     DevBuf lat;                        // latent attention: [slots][Smax][rank]
-    DevBuf gla;                        // HGRN2, gated linear attention: [slots][heads][dim][vdim]
+    DevBuf gla;                        // HGRN2, gated linear attention: [slots][heads][dim][vdim]; matrix memories: [slots][heads][columns][dim]
+    DevBuf run_max;                    // mLSTM: running maxima of the log gates [slots][heads][column blocks]
     DevBuf canon1, canon2;             // sandwich block: the last taps-1 inputs of both sublayers [slots][taps-1][width]
     DevBuf rot_tab, vrot_tab;          // rotation tables (cos, sin) [Smax][pairs] of the queries / keys and of the values
 };
@@ -168,25 +176,28 @@ struct Lin {  // one Linear call on the model's compute dtype
                (bias == nullptr || bias16 != nullptr) && (w_row0 == 0 || (N % 8 == 0 && (w_row0 * (size_t)K) % 8 == 0)) &&
                (reinterpret_cast<uintptr_t>(out) & 15) == 0 && tc_enabled();
     }
-    // a16_ready: A is already there as bf16 rows of pitch K in the model's a16 buffer (the producing kernel wrote them): no cast
+    // whether a product of these sizes can take its input through a dynamic-tanh norm on the way in (a decode step's weight-streaming kernel)
+    bool fuses_norm(int K, int M) const { return linear_fuses_norm(M, K) && (m->seq->d.compute == B2_COMPUTE_F32 || M < tc_min_rows() || !tc_enabled()); }
+    // a16: A is already there as bf16 rows of pitch K (the producing kernel wrote them): no cast. norm: A passes it on the way in (fuses_norm)
     int operator()(const float* A, int64_t lda, const DevBuf& W, int N, int K, float* out, int64_t ldo, int M, int act = LIN_NONE,
                    float alpha = 1.f, int accumulate = 0, const float* bias = nullptr, size_t w_row0 = 0, const void* bias16 = nullptr,
-                   bool a16_ready = false) const {
+                   const void* a16 = nullptr, const DytNorm* norm = nullptr) const {
         LinearArgs a;
         const SeqModel& s = *m->seq;
         a.A = A; a.lda = lda; a.ldw = K; a.w_dtype = s.w_dtype;
         a.W = reinterpret_cast<const char*>(W.p) + w_row0 * (size_t)K * esz(s.w_dtype);
         a.bias = bias; a.out = out; a.ld_out = ldo; a.M = M; a.N = N; a.K = K; a.act = act; a.alpha = alpha; a.accumulate = accumulate;
         a.round_a = s.d.compute == B2_COMPUTE_BF16;
+        if (norm != nullptr) a.norm = *norm;
         // bf16 compute, a portion of a prompt: the tcgen05 GEMM on a bf16 copy of A (weights are stored with their rows
         // padded to a multiple of 8, zero-filled, so N rounds up; the pitch of every projection buffer is a multiple of 8)
         const int Np = (N + 7) / 8 * 8;
         // a block of rows inside a matrix (w_row0 > 0) has no zero rows behind it: then N itself must be a multiple of 8; a bias
         // rides the epilogue as bf16
-        if (tensor_cores(N, K, out, ldo, M, bias, w_row0, bias16)) {
-            if (!a16_ready) B2_TRY(cast_rows_bf16(A, lda, s.a16.p, K, M, K, st));
+        if (norm == nullptr && tensor_cores(N, K, out, ldo, M, bias, w_row0, bias16)) {
+            if (a16 == nullptr) B2_TRY(cast_rows_bf16(A, lda, s.a16.p, K, M, K, st));
             GemmArgs g;
-            g.A = s.a16.p; g.lda = K; g.W = a.W; g.ldw = K; g.out = out; g.ld_out = (int)ldo; g.out_fp32 = 1; g.bias = bias16;
+            g.A = a16 != nullptr ? a16 : s.a16.p; g.lda = K; g.W = a.W; g.ldw = K; g.out = out; g.ld_out = (int)ldo; g.out_fp32 = 1; g.bias = bias16;
             g.M = M; g.N = Np; g.K = K; g.act = ACT_NONE; g.post = act; g.alpha = alpha; g.accumulate = accumulate;
             return gemm_bf16(g, st);
         }
@@ -214,6 +225,14 @@ int attn_nsplit(int rows, int G, int max_seq) {
 }
 
 }  // namespace
+
+// What a sublayer's first product reads: fp32 rows h of pitch width; or (h16) the same rows already rounded to bf16 by the norm that made
+// them; or (norm) the residual stream itself, normed on its way into the product.
+struct SubIn {
+    const float* h = nullptr; const void* h16 = nullptr; const DytNorm* norm = nullptr;
+    SubIn(const float* p) : h(p) {}
+    SubIn() {}
+};
 
 // ------------------------------------------------------------------------------------------------------------------
 // mixers and feed-forwards of the pre-norm and sandwich blocks: they read h [R, width] and write alpha * (their output) to
@@ -335,7 +354,7 @@ static int latent_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeight
 // either pair layout, optionally rotated values, a masked softmax with an optional fixed sink, and a sigmoid output gate per channel or
 // per head. With two maps (differential attention) the projection rows were ordered [map][head][dim] when the tensors were set, so the
 // maps are simply twice the query and key heads over the same value heads, and a head's two outputs are joined after the softmax.
-static int gqa_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeights& W, SeqLayerState& S, const float* h, float* target, float alpha,
+static int gqa_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeights& W, SeqLayerState& S, const SubIn& in, float* target, float alpha,
                      int accumulate, int R, int nseg, cudaStream_t st) {
     SeqModel& s = *m->seq;
     SeqState& state = *kv->seq;
@@ -348,7 +367,7 @@ static int gqa_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeights& 
     const int32_t* row_slot = s.row_slot.as<int32_t>();
     const int32_t* row_pos = s.row_pos.as<int32_t>();
     float* proj = s.proj.as<float>();  // [R, nq | nk | nv | gate]
-    B2_TRY(lin(h, width, W.lproj_w, L.lproj, width, proj, L.lproj_ld, R));
+    B2_TRY(lin(in.h, width, W.lproj_w, L.lproj, width, proj, L.lproj_ld, R, LIN_NONE, 1.f, 0, nullptr, 0, nullptr, in.h16, in.norm));
     float* qkv = proj;
     int64_t ldc = L.lproj_ld;
     if (d.ga_conv >= 1) {
@@ -365,7 +384,8 @@ static int gqa_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeights& 
     rq[0].table = rq[1].table = S.rot_tab.as<float2>(); rq[0].pairs = rq[1].pairs = d.rot_dims / 2;
     rq[0].half = rq[1].half = d.ga_rot_half;
     if (d.ga_qk_norm) { rq[0].norm_w = W.qn_w.as<float>(); rq[1].norm_w = W.kn_w.as<float>(); rq[0].eps = rq[1].eps = s.d.norm_eps; }
-    rq[2].in = qkv + L.nq + L.nk; rq[2].hs_in = dv; rq[2].cache = S.vc.as<float>(); rq[2].heads = G; rq[2].size = dv;
+    rq[0].norm_all = rq[1].norm_all = d.ga_qk_norm == B2_QK_NORM_ALL;
+    rq[2].in = qkv + L.nq + (d.ga_key_values ? 0 : L.nk); rq[2].hs_in = dv; rq[2].cache = S.vc.as<float>(); rq[2].heads = G; rq[2].size = dv;
     rq[2].table = S.vrot_tab.as<float2>(); rq[2].pairs = d.ga_rot_values ? dv / 2 : 0;
     B2_TRY(rotate_rows_multi_f32(rq, 3, st));
     BiasAttnArgs aa;
@@ -374,7 +394,8 @@ static int gqa_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeights& 
     aa.out = s.y.as<float>(); aa.ldo = (int64_t)maps * L.ng;
     aa.H = maps * H; aa.G = maps * G; aa.Gv = maps > 1 ? G : 0; aa.dk = dk; aa.dv = dv; aa.Smax = kv->max_seq; aa.rows = R;
     aa.scale = d.ga_scale;
-    aa.sink_fixed = d.ga_sink != 0; aa.sink_value = d.ga_sink_value;
+    if (d.ga_sink == B2_SINK_HEAD) aa.sink = W.sink.as<float>();
+    else { aa.sink_fixed = d.ga_sink != 0; aa.sink_value = d.ga_sink_value; }
     aa.row_slot = row_slot; aa.row_pos = row_pos;
     aa.nsplit = attn_nsplit(R, maps * G, kv->max_seq);
     aa.tile_rows = max_n;
@@ -439,6 +460,156 @@ static int gla_mixer(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, SeqLayer
     return lin(s.gated.as<float>(), L.pv, W.o_w, width, L.pv, target, width, R, LIN_NONE, alpha, accumulate);
 }
 
+// HGRN2: one fused projection [q | f | v], the recurrence, per-head RMS norm, out-projection.
+static int hgrn2_mixer(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, SeqLayerState& S, const float* h, float* target, float alpha, int accumulate,
+                       int R, int nseg, cudaStream_t st) {
+    SeqModel& s = *m->seq;
+    const b2_seq_layer_desc& d = L.d;
+    const Lin lin{m, st};
+    const int width = s.d.width, H = d.g_heads, dk = d.g_dim, dv = d.g_vdim;
+    float* proj = s.proj.as<float>();  // [R, q | f | v]
+    B2_TRY(lin(h, width, W.qfv_w, L.pproj, width, proj, L.pproj_ld, R));
+    ScanArgs sa;
+    sa.mode = SCAN_HGRN2;
+    sa.q = proj; sa.ldq = L.pproj_ld;
+    sa.decay_in = proj + L.pq; sa.ldd = L.pproj_ld;
+    sa.v = proj + 2 * L.pq; sa.ldv = L.pproj_ld;
+    sa.gate_bias = W.f_b.as<float>(); sa.gate_lower = W.lower.as<float>();
+    sa.state = S.gla.as<float>();
+    sa.y = s.y.as<float>(); sa.ldy = L.pv;
+    sa.heads = H; sa.groups = H; sa.dk = dk; sa.dv = dv;
+    sa.segs = s.segs.as<SeqSeg>(); sa.nseg = nseg;
+    B2_TRY(linear_scan_f32(sa, st));
+    B2_TRY(group_rmsnorm_f32(s.y.as<float>(), L.pv, W.hnorm.as<float>(), 1, s.gated.as<float>(), L.pv, R, L.pv, dv, s.d.norm_eps, st));
+    return lin(s.gated.as<float>(), L.pv, W.o_w, width, L.pv, target, width, R, LIN_NONE, alpha, accumulate);
+}
+
+// The two matrix memories (mLSTM, gated delta rule): one fused projection [q | k | v | gate 1 | gate 2 | g], for the delta rule a convolution with
+// SiLU over q, k, v, the memory with its gates in one kernel, per-head RMS norm with the output gate (straight into the bf16 operand of the
+// out-projection when that runs on the tensor cores), out-projection.
+static int memory_mixer(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, SeqLayerState& S, const SubIn& in, float* target, float alpha, int accumulate,
+                        int R, int nseg, cudaStream_t st) {
+    SeqModel& s = *m->seq;
+    const b2_seq_layer_desc& d = L.d;
+    const Lin lin{m, st};
+    const bool ml = d.type == B2_MIXER_MLSTM;
+    const int width = s.d.width, H = ml ? d.ml_heads : d.dn_heads, dv = ml ? d.ml_vdim : d.dn_vdim;
+    const SeqSeg* segs = s.segs.as<SeqSeg>();
+    float* proj = s.proj.as<float>();
+    B2_TRY(lin(in.h, width, W.mem_w, L.pproj, width, proj, L.pproj_ld, R, LIN_NONE, 1.f, 0, nullptr, 0, nullptr, in.h16, in.norm));
+    const float* gates = proj + L.pq + L.pk + L.pv;
+    const float* qkv = proj;
+    int64_t ld = L.pproj_ld;
+    if (!ml) {
+        B2_TRY(causal_conv_f32(proj, L.pproj_ld, W.conv_w.as<float>(), nullptr, S.conv_tail.as<float>(), s.act.as<float>(), L.conv_ch, L.conv_ch, d.dn_conv,
+                               CONV_SILU, segs, nseg, nseg == 1 ? R : 1, st));
+        qkv = s.act.as<float>();
+        ld = L.conv_ch;
+    }
+    MemoryArgs a;
+    a.mode = ml ? MEM_MLSTM : MEM_DELTA;
+    a.q = qkv; a.k = qkv + L.pq; a.v = qkv + L.pq + L.pk; a.ldq = a.ldk = a.ldv = ld;
+    a.gate1 = gates; a.gate2 = gates + H; a.ldg = L.pproj_ld;
+    a.heads = H; a.dv = dv; a.state = S.gla.as<float>(); a.y = s.y.as<float>(); a.ldy = L.pv; a.segs = segs; a.nseg = nseg;
+    if (ml) {
+        a.kv_heads = H; a.dk = d.ml_dim; a.cap = d.ml_cap; a.bias1 = W.gate1_b.as<float>(); a.bias2 = W.gate2_b.as<float>();
+        a.run_max = S.run_max.as<float>(); a.den = s.den.as<float>();
+    } else {
+        a.kv_heads = d.dn_kv_heads; a.dk = d.dn_dim; a.bias2 = W.dt_bias.as<float>(); a.a_log = W.a_log.as<float>();
+    }
+    a.q_scale = 1.f / sqrtf((float)a.dk);
+    B2_TRY(matrix_memory_f32(a, st));
+    const bool tc = lin.tensor_cores(width, L.pv, target, width, R);
+    B2_TRY(gated_group_rmsnorm_f32(a.y, L.pv, gates + 2 * H, L.pproj_ld, W.mnorm_w.as<float>(), s.gated.as<float>(), L.pv, R, L.pv, dv, 0, s.d.norm_eps, st,
+                                   ml ? 0 : 1, ml ? 1 : 0, a.den, tc ? s.a16.p : nullptr, L.pv));
+    return lin(s.gated.as<float>(), L.pv, W.o_w, width, L.pv, target, width, R, LIN_NONE, alpha, accumulate, nullptr, 0, nullptr, tc ? s.a16.p : nullptr);
+}
+
+// W_down gelu(W_up h) in two steps, so that a parallel block can take the first product before anything joins the residual stream it reads.
+// On the tensor cores the first product's epilogue activates and writes the bf16 rows that the second one reads.
+static bool gelu_on_tensor_cores(const SeqModel& s, const Lin& lin, int ff, float* target, int R) {
+    return ff % 8 == 0 && s.f16.p != nullptr && lin.tensor_cores(ff, s.d.width, s.ff.as<float>(), (ff + 7) / 8 * 8, R) && lin.tensor_cores(s.d.width, ff, target, s.d.width, R);
+}
+static int gelu_up(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, const SubIn& in, float* target, int R, cudaStream_t st) {
+    SeqModel& s = *m->seq;
+    const Lin lin{m, st};
+    const int ff = L.d.ff, width = s.d.width;
+    if (in.norm == nullptr && gelu_on_tensor_cores(s, lin, ff, target, R)) {
+        if (in.h16 == nullptr) B2_TRY(cast_rows_bf16(in.h, width, s.a16.p, width, R, width, st));
+        GemmArgs g;
+        g.A = in.h16 != nullptr ? in.h16 : s.a16.p; g.lda = width; g.W = W.up_w.p; g.ldw = width; g.out = s.f16.p; g.ld_out = ff;
+        g.M = R; g.N = ff; g.K = width; g.act = ACT_GELU_ERF;
+        return gemm_bf16(g, st);
+    }
+    return lin(in.h, width, W.up_w, ff, width, s.ff.as<float>(), (ff + 7) / 8 * 8, R, LIN_GELU, 1.f, 0, nullptr, 0, nullptr, in.h16, in.norm);
+}
+static int gelu_down(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, float* target, float alpha, int accumulate, int R, cudaStream_t st) {
+    SeqModel& s = *m->seq;
+    const Lin lin{m, st};
+    const int ff = L.d.ff, width = s.d.width;
+    const void* f16 = gelu_on_tensor_cores(s, lin, ff, target, R) ? s.f16.p : nullptr;
+    return lin(s.ff.as<float>(), (ff + 7) / 8 * 8, W.down_w, width, ff, target, width, R, LIN_NONE, alpha, accumulate, nullptr, 0, nullptr, f16);
+}
+
+// x <- W_in [x; x0] in front of a pass of the looped block
+static int loop_mix(b2_model* m, float* x, int R, cudaStream_t st) {
+    SeqModel& s = *m->seq;
+    const Lin lin{m, st};
+    const int width = s.d.width;
+    const bool tc = lin.tensor_cores(width, 2 * width, x, width, R);
+    B2_TRY(concat_rows_f32(x, s.x0.as<float>(), s.cat.as<float>(), tc ? s.a16.p : nullptr, R, width, st));
+    return lin(s.cat.as<float>(), 2 * width, s.loop_in, width, 2 * width, x, width, R, LIN_NONE, 1.f, 0, nullptr, 0, nullptr, tc ? s.a16.p : nullptr);
+}
+
+static DytNorm dyt_of(const DevBuf& alpha, const DevBuf& w, const DevBuf& b) { return DytNorm{alpha.as<float>(), w.as<float>(), b.as<float>()}; }
+
+// The norms of a parallel block's two sublayers, both of x. Dynamic tanh: a decode step norms x on its way into the sublayers' first products
+// (nothing is launched here); a prompt portion writes both normed copies in one pass, as the bf16 operands of those products where they
+// run on the tensor cores. n1 / n2 hold what the inputs point to.
+static int parallel_inputs(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, float* x, int R, bool two, int N1, float* target, DytNorm& n1, DytNorm& n2,
+                           SubIn& in1, SubIn& in2, cudaStream_t st) {
+    SeqModel& s = *m->seq;
+    const Lin lin{m, st};
+    const int width = s.d.width;
+    const float eps = s.d.norm_eps;
+    float* xn = s.xn.as<float>();
+    if (s.d.norm_kind != B2_NORM_DYT) {
+        B2_TRY(rms_weight_f32(x, width, nullptr, W.norm1.as<float>(), xn, width, 0, R, width, eps, st));
+        in1 = in2 = SubIn(xn);
+        if (two) {
+            B2_TRY(rms_weight_f32(x, width, nullptr, W.norm2.as<float>(), s.h2.as<float>(), width, 0, R, width, eps, st));
+            in2 = SubIn(s.h2.as<float>());
+        }
+        return 0;
+    }
+    n1 = dyt_of(W.norm1_a, W.norm1, W.norm1_b);
+    if (two) n2 = dyt_of(W.norm2_a, W.norm2, W.norm2_b);
+    // the sublayers whose first product takes a SubIn in all its forms (the others read fp32 rows)
+    const bool mixer_ok = L.d.type == B2_MIXER_GQA_ATTN || L.d.type == B2_MIXER_MLSTM || L.d.type == B2_MIXER_DELTA;
+    const bool ff_ok = L.d.ff == 0 || L.d.ff_kind == B2_FF_GELU;
+    if (lin.fuses_norm(width, R) && mixer_ok && ff_ok) {
+        in1.h = in2.h = x;
+        in1.norm = in2.norm = &n1;
+        if (two) in2.norm = &n2;
+        return 0;
+    }
+    const int Np = (N1 + 7) / 8 * 8;
+    const bool tc1 = mixer_ok && lin.tensor_cores(N1, width, s.proj.as<float>(), Np, R) && (two || L.d.ff == 0);
+    const bool tc2 = two && L.d.ff_kind == B2_FF_GELU && gelu_on_tensor_cores(s, lin, L.d.ff, target, R);
+    DytOut o[2];
+    o[0].norm = n1;
+    if (tc1) { o[0].out16 = s.h1_16.p; in1 = SubIn(xn); in1.h16 = s.h1_16.p; }
+    else { o[0].out = xn; in1 = SubIn(xn); }
+    in2 = in1;
+    if (two) {
+        o[1].norm = n2;
+        in2 = SubIn(s.h2.as<float>());
+        if (tc2) { o[1].out16 = s.h2_16.p; in2.h16 = s.h2_16.p; }
+        else o[1].out = s.h2.as<float>();
+    }
+    return dyt_rows_f32(x, nullptr, o, two ? 2 : 1, R, width, st);
+}
+
 // What a sublayer of a sandwich block reads: the pending sublayer output (weight `post`, in mixout) joins x, x is normed with
 // `norm` into xn, and the input convolution adds to it (a decode step: in the same launch). *h: where the result lies.
 static int sandwich_input(SeqModel& s, const float* post, const DevBuf& norm, const DevBuf& taps_w, DevBuf& tail, int R, int nseg, int max_n,
@@ -492,11 +663,15 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
             B2_TRY(lin(h, width, W.up_w, 2 * ff, width, s.ff.as<float>(), ffl, R));
             if (lin.tensor_cores(width, ff, target, width, R)) {   // the unit writes the bf16 rows that the second product reads
                 B2_TRY(glu_rows_f32(s.ff.as<float>(), ffl, nullptr, 0, R, ff, act, st, s.a16.p, ff));
-                return lin(nullptr, 0, W.down_w, width, ff, target, width, R, LIN_NONE, alpha, accumulate, nullptr, 0, nullptr, true);
+                return lin(nullptr, 0, W.down_w, width, ff, target, width, R, LIN_NONE, alpha, accumulate, nullptr, 0, nullptr, s.a16.p);
             }
             B2_TRY(glu_rows_f32(s.ff.as<float>(), ffl, s.ffa.as<float>(), ff, R, ff, act, st));
         }
         return lin(s.ffa.as<float>(), ff, W.down_w, width, ff, target, width, R, LIN_NONE, alpha, accumulate);
+    }
+    if (d.ff_kind == B2_FF_GELU) {
+        B2_TRY(gelu_up(m, L, W, SubIn(h), target, R, st));
+        return gelu_down(m, L, W, target, alpha, accumulate, R, st);
     }
     if (d.ff_kind != B2_FF_MOE) {
         B2_TRY(lin(h, width, W.up_w, d.ff, width, s.ff.as<float>(), (d.ff + 7) / 8 * 8, R, LIN_RELU_SQ));
@@ -601,7 +776,8 @@ static int seq_forward(b2_model* m, b2_kv* kv, int R, int nseg, int slot, int ct
     float* mix = s.mixout.as<float>();
     const SeqSeg* segs = s.segs.as<SeqSeg>();
     const int max_n = nseg == 1 ? R : 1;  // a prompt portion is one segment of R rows; a decode step is R segments of one row
-    const bool pre = s.d.block == B2_BLOCK_PRE_RMS1, sandwich = s.d.block == B2_BLOCK_SANDWICH_RMS, parallel = s.d.block == B2_BLOCK_PARALLEL_RMS;
+    const bool pre = s.d.block == B2_BLOCK_PRE_RMS1, sandwich = s.d.block == B2_BLOCK_SANDWICH_RMS;
+    const bool parallel = s.d.block == B2_BLOCK_PARALLEL_RMS || s.d.block == B2_BLOCK_PARALLEL2;
     const bool direct = pre || parallel;   // a sublayer's last product adds residual_mult * its output onto x
     const float rm = s.d.residual_mult;
     float* xn = s.xn.as<float>();
@@ -615,18 +791,43 @@ static int seq_forward(b2_model* m, b2_kv* kv, int R, int nseg, int slot, int ct
         // a run that opens a pass of the looped block: x += (the embedding output, from the second pass on) + the pass's vector
         const int pass = s.runs[ri].pass;
         const float* pass_add = pass > 0 ? s.x0.as<float>() : nullptr;
-        const float* pass_vec = pass >= 0 ? s.loop_step.as<float>() + (size_t)pass * width : nullptr;
+        const float* pass_vec = pass >= 0 && !s.d.loop_mix ? s.loop_step.as<float>() + (size_t)pass * width : nullptr;
         if (pre || sandwich || parallel) {
             // pre-norm block: a sublayer reads g * unit_rms(x) and adds residual_mult * its output onto x in its last product.
-            // parallel block: ONE weighted RMS norm per layer; mixer and feed-forward both read it and both add onto x the same way.
+            // parallel block: ONE norm per layer that mixer and feed-forward both read, or one for each; both norms see x in front of the
+            // layer and both sublayers add onto x the same way.
             // sandwich block: a sublayer reads u + conv(u), u = rms_w(x); its output lands in `mix`, and its weighted RMS norm joins x in
             // the same pass that norms x for the next sublayer (`post`: the weight of a sublayer output that has not joined x yet).
             float* target = direct ? x : mix;
             const float alpha = direct ? rm : 1.f;
             const int acc = direct ? 1 : 0;
             const float* h = xn;
+            if (parallel) {
+                if (pass >= 0) B2_TRY(loop_mix(m, x, R, st));
+                const bool two = s.d.block == B2_BLOCK_PARALLEL2 && d.ff > 0, early = d.ff > 0 && d.ff_kind == B2_FF_GELU;
+                DytNorm n1, n2;
+                SubIn in1, in2;
+                B2_TRY(parallel_inputs(m, L, W, x, R, two, L.lproj > 0 ? L.lproj : L.pproj, x, n1, n2, in1, in2, st));
+                if (early) B2_TRY(gelu_up(m, L, W, in2, x, R, st));   // reads x (through its norm) before the mixer's output joins it
+                if (d.type == B2_MIXER_LATENT_ATTN) {
+                    SeqLayerState& KS = d.la_kv_from > 0 ? state.layer[s.runs[ri].kv_run] : S;
+                    B2_TRY(latent_mixer(m, kv, L, W, S, KS, in1.h, x, rm, 1, R, nseg, slot, ctx_end, st));
+                } else if (d.type == B2_MIXER_GQA_ATTN) {
+                    B2_TRY(gqa_mixer(m, kv, L, W, S, in1, x, rm, 1, R, nseg, st));
+                } else if (d.type == B2_MIXER_MLSTM || d.type == B2_MIXER_DELTA) {
+                    B2_TRY(memory_mixer(m, L, W, S, in1, x, rm, 1, R, nseg, st));
+                } else if (d.type == B2_MIXER_GLA) {
+                    B2_TRY(gla_mixer(m, L, W, S, in1.h, x, rm, 1, R, nseg, st));
+                } else {
+                    B2_TRY(hgrn2_mixer(m, L, W, S, in1.h, x, rm, 1, R, nseg, st));
+                }
+                if (early) B2_TRY(gelu_down(m, L, W, x, rm, 1, R, st));
+                else if (d.ff > 0) B2_TRY(seq_feed_forward(m, L, W, in2.h, x, rm, 1, R, st));
+                if (resid_out != nullptr)
+                    B2_CUDA_CHECK(cudaMemcpyAsync(resid_out + ri * (size_t)R * width, x, (size_t)R * width * F4, cudaMemcpyDeviceToDevice, st));
+                continue;
+            }
             if (pre) B2_TRY(rms_scalar_f32(x, nullptr, W.norm1.as<float>(), pass_add, pass_vec, xn, R, width, eps, st));
-            else if (parallel) B2_TRY(rms_weight_f32(x, width, nullptr, W.norm1.as<float>(), xn, width, 0, R, width, eps, st));
             else B2_TRY(sandwich_input(s, post, W.norm1, W.canon1, S.canon1, R, nseg, max_n, st, &h));
             if (d.type == B2_MIXER_LATENT_ATTN) {
                 SeqLayerState& KS = d.la_kv_from > 0 ? state.layer[s.runs[ri].kv_run] : S;
@@ -636,26 +837,11 @@ static int seq_forward(b2_model* m, b2_kv* kv, int R, int nseg, int slot, int ct
             } else if (d.type == B2_MIXER_GLA) {
                 B2_TRY(gla_mixer(m, L, W, S, h, target, alpha, acc, R, nseg, st));
             } else {
-                float* proj = s.proj.as<float>();  // [R, q | f | v]
-                const int H = d.g_heads, dk = d.g_dim, dv = d.g_vdim;
-                B2_TRY(lin(h, width, W.qfv_w, L.pproj, width, proj, L.pproj_ld, R));
-                ScanArgs sa;
-                sa.mode = SCAN_HGRN2;
-                sa.q = proj; sa.ldq = L.pproj_ld;
-                sa.decay_in = proj + L.pq; sa.ldd = L.pproj_ld;
-                sa.v = proj + 2 * L.pq; sa.ldv = L.pproj_ld;
-                sa.gate_bias = W.f_b.as<float>(); sa.gate_lower = W.lower.as<float>();
-                sa.state = S.gla.as<float>();
-                sa.y = s.y.as<float>(); sa.ldy = L.pv;
-                sa.heads = H; sa.groups = H; sa.dk = dk; sa.dv = dv;
-                sa.segs = segs; sa.nseg = nseg;
-                B2_TRY(linear_scan_f32(sa, st));
-                B2_TRY(group_rmsnorm_f32(s.y.as<float>(), L.pv, W.hnorm.as<float>(), 1, s.gated.as<float>(), L.pv, R, L.pv, dv, eps, st));
-                B2_TRY(lin(s.gated.as<float>(), L.pv, W.o_w, width, L.pv, target, width, R, LIN_NONE, alpha, acc));
+                B2_TRY(hgrn2_mixer(m, L, W, S, h, target, alpha, acc, R, nseg, st));
             }
             post = sandwich ? W.norm1_b.as<float>() : nullptr;
             if (d.ff > 0) {
-                h = xn;   // parallel block: the feed-forward reads what the mixer read
+                h = xn;
                 if (pre) B2_TRY(rms_scalar_f32(x, nullptr, W.norm2.as<float>(), nullptr, nullptr, xn, R, width, eps, st));
                 else if (sandwich) B2_TRY(sandwich_input(s, post, W.norm2, W.canon2, S.canon2, R, nseg, max_n, st, &h));
                 B2_TRY(seq_feed_forward(m, L, W, h, target, alpha, acc, R, st));
@@ -769,14 +955,30 @@ static int seq_embed(b2_model* m, b2_kv* kv, const int32_t* tokens, int R, int n
 // rows `index` (null: all) of x -> final norm -> head -> soft-cap: fp32 logits [n, vocab]
 static int seq_head(b2_model* m, const int32_t* index, int n, float* logits, int64_t ld, cudaStream_t st) {
     SeqModel& s = *m->seq;
-    if (s.d.block == B2_BLOCK_PRE_RMS1)
+    const Lin lin{m, st};
+    const DevBuf& head = s.d.tied_head ? s.embed : s.head;
+    const float lscale = s.d.logit_scale != 0.f ? s.d.logit_scale : 1.f;
+    const float* in = s.xn.as<float>();
+    const void* in16 = nullptr;
+    DytNorm dn;
+    if (s.d.norm_kind == B2_NORM_DYT) {
+        DytOut o;
+        o.norm = dn = dyt_of(s.final_a, s.final_w, s.final_b);
+        if (index == nullptr && lin.fuses_norm(s.d.width, n)) {   // a decode step: the rows are normed on their way into the product
+            in = s.x.as<float>();
+        } else {
+            dn.alpha = nullptr;
+            if (lin.tensor_cores(s.d.vocab, s.d.width, logits, ld, n)) o.out16 = const_cast<void*>(in16 = s.a16.p);
+            else o.out = s.xn.as<float>();
+            B2_TRY(dyt_rows_f32(s.x.as<float>(), index, &o, 1, n, s.d.width, st));
+        }
+    } else if (s.d.block == B2_BLOCK_PRE_RMS1)
         B2_TRY(rms_scalar_f32(s.x.as<float>(), index, s.final_w.as<float>(), nullptr, nullptr, s.xn.as<float>(), n, s.d.width, s.d.norm_eps, st));
-    else if (s.d.block == B2_BLOCK_SANDWICH_RMS || s.d.block == B2_BLOCK_PARALLEL_RMS)
+    else if (s.d.block == B2_BLOCK_SANDWICH_RMS || s.d.block == B2_BLOCK_PARALLEL_RMS || s.d.block == B2_BLOCK_PARALLEL2)
         B2_TRY(rms_weight_f32(s.x.as<float>(), s.d.width, index, s.final_w.as<float>(), s.xn.as<float>(), s.d.width, 0, n, s.d.width, s.d.norm_eps, st));
     else
         B2_TRY(layernorm_gather_f32(s.x.as<float>(), index, s.final_w.as<float>(), s.final_b.as<float>(), s.xn.as<float>(), n, s.d.width, s.d.norm_eps, st));
-    const Lin lin{m, st};
-    B2_TRY(lin(s.xn.as<float>(), s.d.width, s.head, s.d.vocab, s.d.width, logits, ld, n, LIN_NONE, s.d.logit_scale != 0.f ? s.d.logit_scale : 1.f));
+    B2_TRY(lin(in, s.d.width, head, s.d.vocab, s.d.width, logits, ld, n, LIN_NONE, lscale, 0, nullptr, 0, nullptr, in16, dn.alpha != nullptr ? &dn : nullptr));
     if (s.d.logit_softcap > 0.f) {
         B2_CHECK_ARG(ld == s.d.vocab, "seq_head: soft-capped logits are contiguous rows");
         B2_TRY(softcap_f32(logits, (size_t)n * s.d.vocab, s.d.logit_softcap, st));
@@ -805,9 +1007,10 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
     SeqModel& s = *m->seq;
     const int width = s.d.width, V = s.d.vocab, WD = s.w_dtype;
     const std::string k(key);
-    if (k == "embed") { B2_TRY(want_shape(key, shape, ndim, V, width)); s.got[k] = 1; return put_tensor(s.embed, WD, (size_t)V * width, 0, ptr, dt, (int64_t)V * width); }
-    if (k == "head") { B2_TRY(want_shape(key, shape, ndim, V, width)); s.got[k] = 1; return put_tensor(s.head, WD, (size_t)((V + 7) / 8 * 8) * width, 0, ptr, dt, (int64_t)V * width); }
-    const bool sandwich = s.d.block == B2_BLOCK_SANDWICH_RMS, parallel = s.d.block == B2_BLOCK_PARALLEL_RMS;
+    if (k == "embed") { B2_TRY(want_shape(key, shape, ndim, V, width)); s.got[k] = 1; return put_tensor(s.embed, WD, (size_t)((V + 7) / 8 * 8) * width, 0, ptr, dt, (int64_t)V * width); }
+    if (k == "head" && !s.d.tied_head) { B2_TRY(want_shape(key, shape, ndim, V, width)); s.got[k] = 1; return put_tensor(s.head, WD, (size_t)((V + 7) / 8 * 8) * width, 0, ptr, dt, (int64_t)V * width); }
+    const bool sandwich = s.d.block == B2_BLOCK_SANDWICH_RMS, parallel2 = s.d.block == B2_BLOCK_PARALLEL2, parallel = s.d.block == B2_BLOCK_PARALLEL_RMS || parallel2;
+    const bool dyt = s.d.norm_kind == B2_NORM_DYT;
     const bool pre = s.d.block == B2_BLOCK_PRE_RMS1 || sandwich || parallel;   // blocks whose layers are made of the mixers / feed-forwards below
     if (k == "final.norm" && s.d.block == B2_BLOCK_PRE_RMS1) { B2_TRY(want_shape(key, shape, ndim, 1)); s.got[k] = 1; return put_tensor(s.final_w, DT_F32, 1, 0, ptr, dt, 1); }
     if (k == "bigram" && s.d.bigram_buckets > 0) {
@@ -815,7 +1018,12 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
         B2_TRY(want_shape(key, shape, ndim, rows, width)); s.got[k] = 1;
         return put_tensor(s.bigram, WD, (size_t)rows * width, 0, ptr, dt, rows * width);
     }
-    if (k == "loop.step" && s.d.loop_times >= 1 && !s.d.loop_plain) {
+    if (k == "loop.in" && s.d.loop_mix) {
+        B2_TRY(want_shape(key, shape, ndim, width, 2 * width)); s.got[k] = 1;
+        return put_tensor(s.loop_in, WD, (size_t)((width + 7) / 8 * 8) * 2 * width, 0, ptr, dt, (int64_t)width * 2 * width);
+    }
+    if (k == "final.norm.alpha" && dyt) { B2_TRY(want_shape(key, shape, ndim, 1)); s.got[k] = 1; return put_tensor(s.final_a, DT_F32, 1, 0, ptr, dt, 1); }
+    if (k == "loop.step" && s.d.loop_times >= 1 && !s.d.loop_plain && !s.d.loop_mix) {
         B2_TRY(want_shape(key, shape, ndim, s.d.loop_times, width)); s.got[k] = 1;
         return put_tensor(s.loop_step, DT_F32, (size_t)s.d.loop_times * width, 0, ptr, dt, (int64_t)s.d.loop_times * width);
     }
@@ -858,6 +1066,13 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
             }
         } else if (parallel) {
             if (r == "norm1") return vec(W.norm1, width);
+            if (r == "norm1.b" && dyt) return vec(W.norm1_b, width);
+            if (r == "norm1.alpha" && dyt) return vec(W.norm1_a, 1);
+            if (parallel2) {   // a layer without feed-forward may carry the second norm all the same: it is not read
+                if (r == "norm2") return vec(W.norm2, width);
+                if (r == "norm2.b" && dyt) return vec(W.norm2_b, width);
+                if (r == "norm2.alpha" && dyt) return vec(W.norm2_a, 1);
+            }
         } else {
             if (r == "norm1") return vec(W.norm1, 1);
             if (r == "norm2" && d.ff > 0) return vec(W.norm2, 1);
@@ -933,9 +1148,11 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
             }
             if (r == "mix.o") return mat(W.o_w, width, L.ng);
             if (d.ga_qk_norm) {
-                if (r == "mix.q.norm") return vec(W.qn_w, d.ga_dim);
-                if (r == "mix.k.norm") return vec(W.kn_w, d.ga_dim);
+                const bool all = d.ga_qk_norm == B2_QK_NORM_ALL;
+                if (r == "mix.q.norm") return vec(W.qn_w, all ? L.nq : d.ga_dim);
+                if (r == "mix.k.norm") return vec(W.kn_w, all ? L.nk : d.ga_dim);
             }
+            if (r == "mix.sink" && d.ga_sink == B2_SINK_HEAD) return vec(W.sink, d.ga_heads);
             if (L.maps > 1) {
                 const char* lam[4] = {"mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"};
                 for (int j = 0; j < 4; ++j)
@@ -957,6 +1174,25 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
             if (r == "mix.a2.b") return vec(W.a2_b, (int64_t)H * dk);
             if (r == "mix.norm") return vec(W.gnorm, dv);
             if (r == "mix.o") return mat(W.o_w, width, (int64_t)H * dv);
+        } else if (d.type == B2_MIXER_MLSTM || d.type == B2_MIXER_DELTA) {
+            // [q | k | v | gate 1 | gate 2 | g]: one matrix, one product (the gates are mLSTM's input / forget gate, the delta rule's write strength /
+            // decay; the output gate comes last)
+            const bool ml = d.type == B2_MIXER_MLSTM;
+            const int H = ml ? d.ml_heads : d.dn_heads, dv = ml ? d.ml_vdim : d.dn_vdim;
+            const char* parts[6] = {"mix.q", "mix.k", "mix.v", ml ? "mix.i" : "mix.b", ml ? "mix.f" : "mix.a", "mix.g"};
+            const int sizes[6] = {L.pq, L.pk, L.pv, H, H, L.pv};
+            int row0 = 0;
+            for (int j = 0; j < 6; ++j) {
+                if (r == parts[j]) return part(W.mem_w, L.pproj, row0, sizes[j], width);
+                if (!ml && j < 3 && r == std::string(parts[j]) + ".conv") return taps_of(W.conv_w, sizes[j], L.conv_ch, row0, d.dn_conv);
+                row0 += sizes[j];
+            }
+            if (r == "mix.norm") return vec(W.mnorm_w, ml ? L.pv : dv);
+            if (r == "mix.o") return mat(W.o_w, width, L.pv);
+            if (ml && r == "mix.i.b") return vec(W.gate1_b, H);
+            if (ml && r == "mix.f.b") return vec(W.gate2_b, H);
+            if (!ml && r == "mix.dt_bias") return vec(W.dt_bias, H);
+            if (!ml && r == "mix.A_log") return vec(W.a_log, H);
         } else if (d.type == B2_MIXER_HGRN2) {
             const int H = d.g_heads, dk = d.g_dim, dv = d.g_vdim;
             if (r == "mix.q") return part(W.qfv_w, L.pproj, 0, L.pq, width);
@@ -1071,11 +1307,16 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
     return -1;
 }
 
-static std::vector<std::string> required_of(const SeqLayerInfo& L, int block, int ctaps) {
-    const bool sandwich = block == B2_BLOCK_SANDWICH_RMS, parallel = block == B2_BLOCK_PARALLEL_RMS;
+static std::vector<std::string> required_of(const SeqLayerInfo& L, const b2_seq_model_desc& md) {
+    const int block = md.block, ctaps = md.input_conv_taps;
+    const bool sandwich = block == B2_BLOCK_SANDWICH_RMS, parallel = block == B2_BLOCK_PARALLEL_RMS, dyt = md.norm_kind == B2_NORM_DYT;
     if (block != B2_BLOCK_POST_LN) {
         std::vector<std::string> v = {"norm1", "mix.o"};
         const b2_seq_layer_desc& d = L.d;
+        if (dyt) {
+            for (const char* n : {"norm1.b", "norm1.alpha"}) v.push_back(n);
+            if (d.ff > 0 && block == B2_BLOCK_PARALLEL2) for (const char* n : {"norm2.b", "norm2.alpha"}) v.push_back(n);
+        }
         if (sandwich) { v.push_back("norm1b"); if (ctaps >= 1) v.push_back("canon1"); }
         if (d.type == B2_MIXER_LATENT_ATTN) {
             for (const char* n : {"mix.uk", "mix.uv"}) v.push_back(n);
@@ -1085,13 +1326,20 @@ static std::vector<std::string> required_of(const SeqLayerInfo& L, int block, in
             if (!d.la_no_sink) v.push_back("mix.sink");
             if (!d.la_no_gate) v.push_back("mix.g");
         } else if (d.type == B2_MIXER_GQA_ATTN) {
-            for (const char* n : {"mix.q", "mix.k", "mix.v"}) v.push_back(n);
+            for (const char* n : {"mix.q", "mix.k"}) v.push_back(n);
+            if (!d.ga_key_values) v.push_back("mix.v");
+            if (d.ga_sink == B2_SINK_HEAD) v.push_back("mix.sink");
             if (L.gw > 0) v.push_back("mix.g");
             if (d.ga_conv >= 1) for (const char* n : {"mix.q.conv", "mix.k.conv", "mix.v.conv"}) v.push_back(n);
             if (d.ga_qk_norm) for (const char* n : {"mix.q.norm", "mix.k.norm"}) v.push_back(n);
             if (L.maps > 1) for (const char* n : {"mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"}) v.push_back(n);
         } else if (d.type == B2_MIXER_GLA) {
             for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.g", "mix.a1", "mix.a2", "mix.a2.b", "mix.norm"}) v.push_back(n);
+        } else if (d.type == B2_MIXER_MLSTM) {
+            for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.g", "mix.i", "mix.i.b", "mix.f", "mix.f.b", "mix.norm"}) v.push_back(n);
+        } else if (d.type == B2_MIXER_DELTA) {
+            for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.q.conv", "mix.k.conv", "mix.v.conv", "mix.g", "mix.a", "mix.b", "mix.A_log", "mix.dt_bias", "mix.norm"})
+                v.push_back(n);
         } else for (const char* n : {"mix.q", "mix.f", "mix.f.b", "mix.lower", "mix.v", "mix.norm"}) v.push_back(n);
         if (L.d.ff > 0) {
             if (!parallel) v.push_back("norm2");
@@ -1129,15 +1377,19 @@ int seq_finalize(b2_model* m) {
     std::string missing;
     const bool sandwich = s.d.block == B2_BLOCK_SANDWICH_RMS;
     const bool pre = s.d.block != B2_BLOCK_POST_LN;
-    std::vector<std::string> top = {"embed", "head", "final.norm"};
-    if (!pre) top.push_back("final.norm.b");
+    std::vector<std::string> top = {"embed", "final.norm"};
+    const bool dyt = s.d.norm_kind == B2_NORM_DYT;
+    if (!s.d.tied_head) top.push_back("head");
+    if (!pre || dyt) top.push_back("final.norm.b");
+    if (dyt) top.push_back("final.norm.alpha");
+    if (s.d.loop_mix) top.push_back("loop.in");
     if (s.d.bigram_buckets > 0) top.push_back("bigram");
-    if (s.d.loop_times >= 1 && !s.d.loop_plain) top.push_back("loop.step");
+    if (s.d.loop_times >= 1 && !s.d.loop_plain && !s.d.loop_mix) top.push_back("loop.step");
     for (const std::string& n : top)
         if (!s.got.count(n) && missing.size() < 600) { missing += n; missing += ' '; }
     for (size_t i = 0; i < s.layers.size(); ++i) {
         if (s.layers[i].src != (int)i) continue;
-        for (const std::string& n : required_of(s.layers[i], s.d.block, s.d.input_conv_taps))
+        for (const std::string& n : required_of(s.layers[i], s.d))
             if (!s.w[i].got.count(n) && missing.size() < 600) missing += "l" + std::to_string(i) + "." + n + " ";
     }
     if (!missing.empty()) {
@@ -1158,7 +1410,8 @@ int seq_finalize(b2_model* m) {
     const int width = s.d.width;
     int pw = 1, aw = 1, yw = 1, rw = 1, kw = 1, fw = 1;
     int latw = 0, moe_top = 0, moe_e = 0, moe_ff = 0;
-    bool glu = false;
+    int den_w = 0;
+    bool glu = false, gelu = false;
     for (const SeqLayerInfo& L : s.layers) {
         if (L.d.type == B2_MIXER_MAMBA2) {
             pw = std::max(pw, L.dproj_ld); aw = std::max(aw, L.conv_ch); yw = std::max(yw, L.inner);
@@ -1168,6 +1421,9 @@ int seq_finalize(b2_model* m) {
             pw = std::max(pw, L.lproj_ld); yw = std::max(yw, L.maps * L.ng); aw = std::max(aw, L.conv_ch);
         } else if (L.d.type == B2_MIXER_GLA) {
             pw = std::max(pw, L.pproj_ld); yw = std::max(yw, L.pv); rw = std::max(rw, L.pq);
+        } else if (L.d.type == B2_MIXER_MLSTM || L.d.type == B2_MIXER_DELTA) {
+            pw = std::max(pw, L.pproj_ld); yw = std::max(yw, L.pv); aw = std::max(aw, L.conv_ch);
+            if (L.d.type == B2_MIXER_MLSTM) den_w = std::max(den_w, L.d.ml_heads);
         } else {
             pw = std::max(pw, L.pproj_ld); yw = std::max(yw, L.pv);
             if (L.d.type == B2_MIXER_LATENT_ATTN) {
@@ -1176,6 +1432,7 @@ int seq_finalize(b2_model* m) {
             }
         }
         fw = std::max(fw, (L.d.ff + 7) / 8 * 8);
+        if (L.d.ff > 0 && L.d.ff_kind == B2_FF_GELU) gelu = true;
         if (L.d.ff > 0 && L.d.ff_kind == B2_FF_CLAMP_GLU) { fw = std::max(fw, (2 * L.d.ff + 7) / 8 * 8); glu = true; }
         if (L.d.ff > 0 && L.d.ff_kind == B2_FF_MOE) {
             fw = std::max(fw, (2 * L.d.moe_shared_ff + 7) / 8 * 8);
@@ -1199,7 +1456,17 @@ int seq_finalize(b2_model* m) {
     B2_TRY(s.xn.alloc(R * width * F4));
     if (pre) B2_TRY(s.ffa.alloc(R * fw * F4));
     if (sandwich && s.d.input_conv_taps >= 1) B2_TRY(s.hin.alloc(R * width * F4));
-    if (s.d.loop_times > 1 && !s.d.loop_plain) B2_TRY(s.x0.alloc(R * width * F4));
+    if (s.d.loop_mix || (s.d.loop_times > 1 && !s.d.loop_plain)) B2_TRY(s.x0.alloc(R * width * F4));
+    if (s.d.loop_mix) B2_TRY(s.cat.alloc(R * 2 * width * F4));
+    if (s.d.block == B2_BLOCK_PARALLEL2) B2_TRY(s.h2.alloc(R * width * F4));
+    if (den_w > 0) B2_TRY(s.den.alloc(R * den_w * F4));
+    if (s.d.compute == B2_COMPUTE_BF16) {
+        if (dyt) {
+            B2_TRY(s.h1_16.alloc(R * width * 2));
+            B2_TRY(s.h2_16.alloc(R * width * 2));
+        }
+        if (gelu) B2_TRY(s.f16.alloc(R * fw * 2));
+    }
     if (glu && moe_e == 0) {   // the one-row grouped product of a decode step reads its group (always 0) from here
         B2_TRY(s.zero_idx.alloc(64 * 4));
         B2_CUDA_CHECK(cudaMemset(s.zero_idx.p, 0, 64 * 4));
@@ -1230,7 +1497,7 @@ int seq_finalize(b2_model* m) {
         if (s.d.compute == B2_COMPUTE_BF16) B2_TRY(s.moe_a16.alloc(P * (size_t)(width + moe_ff) * 2));
     }
     {
-        int kmax = width;
+        int kmax = s.d.loop_mix ? 2 * width : width;
         for (const SeqLayerInfo& L : s.layers)
             kmax = std::max(kmax, std::max(std::max(std::max(L.inner, L.ng), std::max(L.rn, L.d.ff)), std::max(std::max(L.pv, std::max(L.lrow, L.d.la_q_rank)), std::max(L.d.la_dim, L.d.moe_shared_ff))));
         s.a16_w = (kmax + 7) / 8 * 8;
@@ -1253,12 +1520,13 @@ void seq_model_free(b2_model* m) {
                         &W.lproj_w, &W.rel, &W.lo_w, &W.mu, &W.r_w, &W.k_w, &W.v_w, &W.g_w, &W.w1, &W.w2, &W.w0, &W.bonus, &W.rnorm, &W.ro_w,
                         &W.up_w, &W.down_w, &W.qdg_w, &W.dkv_norm, &W.uk_w, &W.ukT, &W.uv_w, &W.sink, &W.qfv_w, &W.f_b, &W.lower, &W.hnorm, &W.up_b, &W.down_b,
                         &W.down_b16, &W.act_coef, &W.router_w, &W.egu_w, &W.ed_w, &W.sgu_w, &W.sd_w, &W.canon1, &W.canon2, &W.dq_norm, &W.uq_w, &W.ukx_w,
-                        &W.qn_w, &W.kn_w, &W.lam4, &W.gla_w, &W.a2_w, &W.a2_b, &W.gnorm};
+                        &W.qn_w, &W.kn_w, &W.lam4, &W.gla_w, &W.a2_w, &W.a2_b, &W.gnorm, &W.norm1_a, &W.norm2_a, &W.mem_w, &W.mnorm_w, &W.gate1_b, &W.gate2_b};
         for (DevBuf* b : bs) b->free();
     }
     DevBuf* bs[] = {&s.embed, &s.head, &s.final_w, &s.final_b, &s.x, &s.proj, &s.act, &s.y, &s.gated, &s.mixout, &s.mixes, &s.rp, &s.wl1, &s.wlog,
                     &s.ff, &s.xn, &s.tok, &s.want, &s.segs, &s.row_slot, &s.row_pos, &s.a16, &s.bigram, &s.loop_step, &s.x0, &s.qabs, &s.olat, &s.ffa,
-                    &s.rlogit, &s.moe_idx, &s.moe_w, &s.moe_pos, &s.moe_src, &s.moe_tile, &s.moe_h, &s.moe_a, &s.moe_y, &s.moe_a16, &s.zero_idx, &s.hin};
+                    &s.rlogit, &s.moe_idx, &s.moe_w, &s.moe_pos, &s.moe_src, &s.moe_tile, &s.moe_h, &s.moe_a, &s.moe_y, &s.moe_a16, &s.zero_idx, &s.hin, &s.final_a, &s.loop_in, &s.cat,
+                    &s.h2, &s.h1_16, &s.h2_16, &s.f16, &s.den};
     for (DevBuf* b : bs) b->free();
     delete m->seq;
     m->seq = nullptr;
@@ -1286,6 +1554,8 @@ int64_t seq_kv_bytes(const b2_model* m, int B, int Smax) {
         else if (d.type == B2_MIXER_LATENT_ATTN) n += d.la_kv_from == 0 ? (int64_t)B * Smax * L.lrow : 0;
         else if (d.type == B2_MIXER_GQA_ATTN) n += (int64_t)B * d.ga_kv_heads * Smax * (L.maps * d.ga_dim + d.ga_vdim) + (int64_t)B * std::max(0, d.ga_conv - 1) * L.conv_ch;
         else if (d.type == B2_MIXER_GLA) n += (int64_t)B * d.gl_heads * d.gl_dim * d.gl_vdim;
+        else if (d.type == B2_MIXER_MLSTM) n += (int64_t)B * d.ml_heads * ((int64_t)d.ml_dim * (d.ml_vdim + 1) + mem_blocks(d.ml_vdim + 1));
+        else if (d.type == B2_MIXER_DELTA) n += (int64_t)B * d.dn_heads * d.dn_dim * d.dn_vdim + (int64_t)B * (d.dn_conv - 1) * L.conv_ch;
         else n += (int64_t)B * d.g_heads * d.g_dim * d.g_vdim;
         if (m->seq->d.block == B2_BLOCK_SANDWICH_RMS && m->seq->d.input_conv_taps > 1)
             n += (int64_t)B * (m->seq->d.input_conv_taps - 1) * m->seq->d.width * (d.ff > 0 ? 2 : 1);
@@ -1318,7 +1588,7 @@ int seq_kv_alloc(b2_kv* kv) {
         if (d.rot_dims >= 2 && (d.type == B2_MIXER_GQA_ATTN || (d.type == B2_MIXER_LATENT_ATTN && d.la_rot_dim > 0))) {
             RotaryDesc rdesc;
             rdesc.dims = d.rot_dims; rdesc.base = d.rot_base; rdesc.factor = d.rot_factor; rdesc.original = d.rot_original; rdesc.fast = d.rot_fast;
-            rdesc.slow = d.rot_slow;
+            rdesc.slow = d.rot_slow; rdesc.scaling = d.rot_scaling;
             B2_TRY(S.rot_tab.alloc(Smax * (d.rot_dims / 2) * sizeof(float2)));
             B2_TRY(rotary_table_build(rdesc, (int)Smax, S.rot_tab.as<float2>()));
         }
@@ -1352,6 +1622,18 @@ int seq_kv_alloc(b2_kv* kv) {
         } else if (d.type == B2_MIXER_GLA) {
             B2_TRY(S.gla.alloc(B * d.gl_heads * d.gl_dim * d.gl_vdim * F4));
             cudaMemset(S.gla.p, 0, S.gla.bytes);
+        } else if (d.type == B2_MIXER_MLSTM) {
+            B2_TRY(S.gla.alloc(B * d.ml_heads * d.ml_dim * (d.ml_vdim + 1) * F4));
+            B2_TRY(S.run_max.alloc(B * d.ml_heads * mem_blocks(d.ml_vdim + 1) * F4));
+            cudaMemset(S.gla.p, 0, S.gla.bytes);
+            cudaMemset(S.run_max.p, 0, S.run_max.bytes);
+        } else if (d.type == B2_MIXER_DELTA) {
+            B2_TRY(S.gla.alloc(B * d.dn_heads * d.dn_dim * d.dn_vdim * F4));
+            cudaMemset(S.gla.p, 0, S.gla.bytes);
+            if (d.dn_conv > 1) {
+                B2_TRY(S.conv_tail.alloc(B * (d.dn_conv - 1) * L.conv_ch * F4));
+                cudaMemset(S.conv_tail.p, 0, S.conv_tail.bytes);
+            }
         } else if (d.type == B2_MIXER_MAMBA2) {
             B2_TRY(S.ssm.alloc(B * d.m_heads * d.m_state * d.m_vdim * F4));
             B2_TRY(S.conv_tail.alloc(std::max<size_t>(1, B * (d.m_conv - 1) * L.conv_ch) * F4));
@@ -1390,7 +1672,7 @@ int seq_kv_alloc(b2_kv* kv) {
 void seq_kv_free(b2_kv* kv) {
     if (kv->seq == nullptr) return;
     for (SeqLayerState& S : kv->seq->layer) {
-        DevBuf* bs[] = {&S.ssm, &S.conv_tail, &S.kc, &S.vc, &S.bucket_of, &S.wkv, &S.prev, &S.lat, &S.gla, &S.canon1, &S.canon2, &S.rot_tab, &S.vrot_tab};
+        DevBuf* bs[] = {&S.ssm, &S.conv_tail, &S.kc, &S.vc, &S.bucket_of, &S.wkv, &S.prev, &S.lat, &S.gla, &S.run_max, &S.canon1, &S.canon2, &S.rot_tab, &S.vrot_tab};
         for (DevBuf* b : bs) b->free();
     }
     kv->seq->last_tok.free();
@@ -1417,7 +1699,10 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
     B2_CHECK_ARG(d.compute == B2_COMPUTE_BF16 || d.compute == B2_COMPUTE_F32, "b2_seq_model_create: unknown compute mode %d", d.compute);
     B2_CHECK_ARG(d.max_batch >= 1 && d.max_rows >= 1, "b2_seq_model_create: bad workspace sizing");
     B2_CHECK_ARG(d.norm_eps >= 0.f, "b2_seq_model_create: negative eps");
-    B2_CHECK_ARG(d.block >= B2_BLOCK_POST_LN && d.block <= B2_BLOCK_PARALLEL_RMS, "b2_seq_model_create: unknown block form %d", d.block);
+    B2_CHECK_ARG(d.block >= B2_BLOCK_POST_LN && d.block <= B2_BLOCK_PARALLEL2, "b2_seq_model_create: unknown block form %d", d.block);
+    const bool par = d.block == B2_BLOCK_PARALLEL_RMS || d.block == B2_BLOCK_PARALLEL2;
+    B2_CHECK_ARG(d.norm_kind == B2_NORM_RMS || (d.norm_kind == B2_NORM_DYT && par), "b2_seq_model_create: norm kind %d does not go with block form %d", d.norm_kind, d.block);
+    B2_CHECK_ARG(!d.loop_mix || (par && d.loop_times >= 1), "b2_seq_model_create: the input mix belongs to a looped block of a parallel-block model");
     B2_CHECK_ARG(d.embed_scale == 0.f || d.bigram_buckets == 0, "b2_seq_model_create: a scaled embedding does not go with the hashed bigram rows");
     B2_CHECK_ARG(d.input_conv_taps >= 0 && d.input_conv_taps <= 16, "b2_seq_model_create: 0..16 taps of the input convolution");
     B2_CHECK_ARG(d.input_conv_taps == 0 || d.block == B2_BLOCK_SANDWICH_RMS, "b2_seq_model_create: the input convolution belongs to the sandwich block");
@@ -1494,6 +1779,9 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
         } else if (l.type == B2_MIXER_GQA_ATTN) {
             if (l.ga_heads < 1 || l.ga_kv_heads < 1 || l.ga_heads % l.ga_kv_heads) why = "attention: heads must be a positive multiple of kv_heads";
             else if (l.ga_dim < 1 || l.ga_dim > 512 || l.ga_vdim < 1 || l.ga_vdim > 512) why = "attention: head sizes 1..512";
+            else if (l.ga_key_values && (l.ga_vdim != l.ga_dim || l.ga_maps == 2 || l.ga_conv > 0)) why = "attention: keys that serve as values have the values' size, one map and no convolution";
+            else if (l.ga_sink < B2_SINK_NONE || l.ga_sink > B2_SINK_HEAD || l.ga_qk_norm < B2_QK_NORM_NONE || l.ga_qk_norm > B2_QK_NORM_ALL) why = "attention: unknown sink or q / k norm";
+            else if (l.ga_sink == B2_SINK_HEAD && l.ga_maps == 2) why = "attention: two maps take no learned sinks";
             else if (l.ga_conv < 0 || l.ga_conv > 16) why = "attention: 0..16 convolution taps";
             else if (l.rot_dims < 0 || l.rot_dims > l.ga_dim || (l.rot_dims > 0 && !(l.rot_base > 0.f))) why = "attention: rotated dimensions within a head, positive base";
             else if (l.rot_factor > 0.f && !(l.rot_original > 0.f && l.rot_fast > 0.f && l.rot_slow > 0.f && l.rot_base > 1.f)) why = "rotation: scaled frequencies need original, fast and slow";
@@ -1505,7 +1793,7 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
             else if (l.ga_gate < B2_GATE_CHANNEL || l.ga_gate > B2_GATE_NONE) why = "attention: unknown output gate";
             else if (l.ga_rot_half && l.rot_dims % 2) why = "attention: the half layout rotates an even number of dimensions";
             L.maps = l.ga_maps == 2 ? 2 : 1;
-            L.nq = L.maps * l.ga_heads * l.ga_dim; L.nk = L.maps * l.ga_kv_heads * l.ga_dim; L.nv = l.ga_kv_heads * l.ga_vdim; L.ng = l.ga_heads * l.ga_vdim;
+            L.nq = L.maps * l.ga_heads * l.ga_dim; L.nk = L.maps * l.ga_kv_heads * l.ga_dim; L.nv = l.ga_key_values ? 0 : l.ga_kv_heads * l.ga_vdim; L.ng = l.ga_heads * l.ga_vdim;
             L.gw = l.ga_gate == B2_GATE_CHANNEL ? L.ng : l.ga_gate == B2_GATE_HEAD ? l.ga_heads : 0;
             L.lproj = L.nq + L.nk + L.nv + L.gw;
             L.lproj_ld = (L.lproj + 7) / 8 * 8;
@@ -1521,10 +1809,26 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
             L.pq = l.gl_heads * l.gl_dim; L.pv = l.gl_heads * l.gl_vdim;
             L.pproj = 2 * L.pq + 2 * L.pv + l.gl_rank;
             L.pproj_ld = (L.pproj + 7) / 8 * 8;
+        } else if (l.type == B2_MIXER_MLSTM) {
+            if (l.ml_heads < 1 || l.ml_dim < 1 || l.ml_dim > 256 || l.ml_vdim < 1) why = "mlstm: heads, dim 1..256, vdim";
+            else if (!(l.ml_cap > 0.f)) why = "mlstm: the gates' cap must be positive";
+            L.pq = L.pk = l.ml_heads * l.ml_dim; L.pv = l.ml_heads * l.ml_vdim;
+            L.pproj = L.pq + L.pk + 2 * L.pv + 2 * l.ml_heads;
+            L.pproj_ld = (L.pproj + 7) / 8 * 8;
+        } else if (l.type == B2_MIXER_DELTA) {
+            if (l.dn_heads < 1 || l.dn_kv_heads < 1 || l.dn_heads % l.dn_kv_heads) why = "delta rule: heads must be a positive multiple of kv_heads";
+            else if (l.dn_dim < 1 || l.dn_dim > 256 || l.dn_vdim < 1) why = "delta rule: dim 1..256, vdim";
+            else if (l.dn_conv < 1 || l.dn_conv > 16) why = "delta rule: 1..16 convolution taps";
+            L.pq = L.pk = l.dn_kv_heads * l.dn_dim; L.pv = l.dn_heads * l.dn_vdim;
+            L.pproj = L.pq + L.pk + 2 * L.pv + 2 * l.dn_heads;
+            L.pproj_ld = (L.pproj + 7) / 8 * 8;
+            L.conv_ch = L.pq + L.pk + L.pv;
         } else {
             why = "unknown mixer type";
         }
-        const bool pre_mixer = l.type == B2_MIXER_LATENT_ATTN || l.type == B2_MIXER_HGRN2 || l.type == B2_MIXER_GQA_ATTN || l.type == B2_MIXER_GLA;
+        const bool pre_mixer = l.type == B2_MIXER_LATENT_ATTN || l.type == B2_MIXER_HGRN2 || l.type == B2_MIXER_GQA_ATTN || l.type == B2_MIXER_GLA || l.type == B2_MIXER_MLSTM || l.type == B2_MIXER_DELTA;
+        if (why == nullptr && (l.type == B2_MIXER_MLSTM || l.type == B2_MIXER_DELTA) && !par) why = "matrix memories need a parallel block";
+        if (why == nullptr && (l.rot_scaling < B2_ROT_YARN || l.rot_scaling > B2_ROT_BANDS)) why = "rotation: unknown scaling";
         if (why == nullptr && pre_mixer != (d.block != B2_BLOCK_POST_LN)) why = "this mixer does not go with the model's block form";
         if (why == nullptr && l.ff > 0) {
             if (l.ff_kind != B2_FF_RELU_SQ && d.block == B2_BLOCK_POST_LN) why = "this feed-forward needs a pre-norm or sandwich block";
@@ -1535,7 +1839,7 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
                 else if (l.moe_score < 0 || l.moe_score > 1 || l.moe_group_score < 0 || l.moe_group_score > 1 || l.moe_act < 0 || l.moe_act > 1) why = "moe: unknown score, group score or activation";
             } else if (l.ff_kind == B2_FF_CLAMP_GLU) {
                 if (l.ff_limit < 0.f) why = "gated feed-forward: negative limit";
-            } else if (l.ff_kind != B2_FF_RELU_SQ && l.ff_kind != B2_FF_POLYNORM) why = "unknown feed-forward kind";
+            } else if (l.ff_kind != B2_FF_RELU_SQ && l.ff_kind != B2_FF_POLYNORM && l.ff_kind != B2_FF_GELU) why = "unknown feed-forward kind";
         }
         if (why == nullptr && L.src != i) {
             b2_seq_layer_desc a = l, b = s->layers[L.src].d;
@@ -1559,7 +1863,7 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
         for (int i = 0; i < d.n_layers; ++i) {
             if (looped && i == d.loop_start) {
                 for (int t = 0; t < d.loop_times; ++t)
-                    for (int j = d.loop_start; j < d.loop_stop; ++j) s->runs.push_back(SeqRun{j, (j == d.loop_start && !d.loop_plain) ? t : -1, -1});
+                    for (int j = d.loop_start; j < d.loop_stop; ++j) s->runs.push_back(SeqRun{j, (j == d.loop_start && (!d.loop_plain || d.loop_mix)) ? t : -1, -1});
                 i = d.loop_stop - 1;
             } else {
                 s->runs.push_back(SeqRun{i, -1, -1});

@@ -78,7 +78,10 @@ class SeqLayerDesc(_c.Structure):
                 ("ga_maps", _c.c_int32), ("ga_diff", _c.c_float), ("ga_qk_norm", _c.c_int32), ("ga_rot_half", _c.c_int32),
                 ("ga_gate", _c.c_int32), ("mask_keep", _c.c_int32),
                 ("gl_heads", _c.c_int32), ("gl_dim", _c.c_int32), ("gl_vdim", _c.c_int32), ("gl_rank", _c.c_int32), ("gl_tau", _c.c_float),
-                ("ff_limit", _c.c_float), ("ff_act_slope", _c.c_float)]
+                ("ff_limit", _c.c_float), ("ff_act_slope", _c.c_float),
+                ("ga_key_values", _c.c_int32), ("rot_scaling", _c.c_int32),
+                ("ml_heads", _c.c_int32), ("ml_dim", _c.c_int32), ("ml_vdim", _c.c_int32), ("ml_cap", _c.c_float),
+                ("dn_heads", _c.c_int32), ("dn_kv_heads", _c.c_int32), ("dn_dim", _c.c_int32), ("dn_vdim", _c.c_int32), ("dn_conv", _c.c_int32)]
 
 
 class SeqModelDesc(_c.Structure):
@@ -88,12 +91,17 @@ class SeqModelDesc(_c.Structure):
                 ("block", _c.c_int32), ("residual_mult", _c.c_float), ("logit_softcap", _c.c_float),
                 ("bigram_buckets", _c.c_int32), ("bigram_mul_prev", _c.c_int32), ("bigram_mul_cur", _c.c_int32),
                 ("loop_start", _c.c_int32), ("loop_stop", _c.c_int32), ("loop_times", _c.c_int32),
-                ("logit_scale", _c.c_float), ("input_conv_taps", _c.c_int32), ("embed_scale", _c.c_float), ("loop_plain", _c.c_int32)]
+                ("logit_scale", _c.c_float), ("input_conv_taps", _c.c_int32), ("embed_scale", _c.c_float), ("loop_plain", _c.c_int32),
+                ("norm_kind", _c.c_int32), ("tied_head", _c.c_int32), ("loop_mix", _c.c_int32)]
 
 
-MIXER_MAMBA2, MIXER_PARALLEL, MIXER_LATENT_ATTN, MIXER_HGRN2, MIXER_GQA_ATTN, MIXER_GLA = 1, 2, 3, 4, 5, 6
-FF_RELU_SQ, FF_POLYNORM, FF_MOE, FF_CLAMP_GLU = 0, 1, 2, 3
-BLOCK_POST_LN, BLOCK_PRE_RMS1, BLOCK_SANDWICH_RMS, BLOCK_PARALLEL_RMS = 0, 1, 2, 3
+MIXER_MAMBA2, MIXER_PARALLEL, MIXER_LATENT_ATTN, MIXER_HGRN2, MIXER_GQA_ATTN, MIXER_GLA, MIXER_MLSTM, MIXER_DELTA = 1, 2, 3, 4, 5, 6, 7, 8
+FF_RELU_SQ, FF_POLYNORM, FF_MOE, FF_CLAMP_GLU, FF_GELU = 0, 1, 2, 3, 4
+BLOCK_POST_LN, BLOCK_PRE_RMS1, BLOCK_SANDWICH_RMS, BLOCK_PARALLEL_RMS, BLOCK_PARALLEL2 = 0, 1, 2, 3, 4
+NORM_RMS, NORM_DYT = 0, 1
+QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_ALL = 0, 1, 2
+SINK_NONE, SINK_FIXED, SINK_HEAD = 0, 1, 2
+ROT_YARN, ROT_BANDS = 0, 1
 GATE_CHANNEL, GATE_HEAD, GATE_NONE = 0, 1, 2
 MASK_CAUSAL, MASK_WINDOW, MASK_CHUNK = 0, 1, 2
 MOE_SCORE_SIGMOID, MOE_SCORE_SOFTMAX = 0, 1

@@ -13,15 +13,17 @@ MODEL_REGISTRY = {
     "Pefivik": ("language_model.pefivik", "PefivikForCausalLM"),
     "Fezuzen": ("language_model.fezuzen", "FezuzenForCausalLM"),
     "Sofopel": ("language_model.sofopel", "SofopelForCausalLM"),
+    "Ramosun": ("language_model.ramosun", "RamosunForCausalLM"),
 }
 _LAZY = {"LlavaLlamaForCausalLM": "language_model.llava_llama", "LlavaConfig": "language_model.llava_llama",
          "KatadraForCausalLM": "language_model.katadra", "KatadraConfig": "language_model.katadra",
          "PefivikForCausalLM": "language_model.pefivik", "PefivikConfig": "language_model.pefivik",
          "FezuzenForCausalLM": "language_model.fezuzen", "FezuzenConfig": "language_model.fezuzen",
-         "SofopelForCausalLM": "language_model.sofopel", "SofopelConfig": "language_model.sofopel"}
+         "SofopelForCausalLM": "language_model.sofopel", "SofopelConfig": "language_model.sofopel",
+         "RamosunForCausalLM": "language_model.ramosun", "RamosunConfig": "language_model.ramosun"}
 
 __all__ = ["LlavaConfig", "LlavaLlamaForCausalLM", "KatadraConfig", "KatadraForCausalLM", "PefivikConfig", "PefivikForCausalLM", "FezuzenConfig",
-           "FezuzenForCausalLM", "SofopelConfig", "SofopelForCausalLM", "MODEL_REGISTRY",
+           "FezuzenForCausalLM", "SofopelConfig", "SofopelForCausalLM", "RamosunConfig", "RamosunForCausalLM", "MODEL_REGISTRY",
            "model_class_for"]
 
 
