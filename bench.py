@@ -55,11 +55,11 @@ def parse_args():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-configs", action="store_true", help="skip the side measurements of the other BASELINE configs")
-    ap.add_argument("--arch", default="llava", choices=["llava", "katadra", "pefivik", "fezuzen", "sofopel"],
+    ap.add_argument("--arch", default="llava", choices=["llava", "katadra", "pefivik", "fezuzen", "sofopel", "ramosun"],
                     help="katadra: prefill / decode throughput of the layer-list decoder beside the LLaMA decoder of equal width, "
                          "depth and parameter count (random weights); the default workload and its JSON line are unchanged")
-    ap.add_argument("--widths", default="2048,4096", help="--arch katadra / pefivik / fezuzen / sofopel: model widths to measure")
-    ap.add_argument("--ctx", type=int, default=2048, help="--arch katadra / pefivik / fezuzen / sofopel: prompt length")
+    ap.add_argument("--widths", default="2048,4096", help="--arch katadra / pefivik / fezuzen / sofopel / ramosun: model widths to measure")
+    ap.add_argument("--ctx", type=int, default=2048, help="--arch katadra / pefivik / fezuzen / sofopel / ramosun: prompt length")
     return ap.parse_args()
 
 
@@ -1025,6 +1025,77 @@ def run_sofopel(args):
     print(json.dumps(out))
 
 
+def ramosun_config(width, ctx):
+    """Four parallel-block layers of the sizes a model of this width would have: window attention (heads of 128 whose values are the keys,
+    four query heads per key/value head, a norm over the whole projection, banded frequency scaling, a window of half the prompt,
+    learned sinks), gated delta rule (value heads of 128, two per q / k head of 128, 4-tap convolutions), mLSTM (keys of 128, values of
+    256) and window attention again, each beside a GELU feed-forward of 3.75 x width (two matrices: the parameters of Sofopel's three
+    of 2.5 x width); the block runs as ONE pass of a loop, so its input mix is in the numbers."""
+    heads = width // 128
+    rot = {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "mask": {"size": ctx // 2}, "rot": rot,
+                                          "scale": 128 ** -0.5}}
+    dlt = {"type": "delta", "mixer": {"heads": heads, "kv_heads": max(1, heads // 2), "dim": 128, "vdim": 128, "conv": 4}}
+    mls = {"type": "mlstm", "mixer": {"heads": max(1, width // 256), "dim": 128, "vdim": 256, "gate_cap": 15.0}}
+    mlp = {"kind": "dense", "ff": 15 * width // 4}
+    return {"architecture": "Ramosun", "width": width, "vocab": 32000, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "loop": {"start": 0, "stop": 4, "times": 1},
+            "layers": [dict(att, mlp=mlp), dict(dlt, mlp=mlp), dict(mls, mlp=mlp), dict(att, mlp=mlp)]}
+
+
+def ramosun_params(cfg):
+    """(matmul parameters a token multiplies with, function B -> parameters a decode step of B slots reads)"""
+    W = cfg["width"]
+    n = cfg["vocab"] * W + 2 * W * W
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        H, dk, dv = m["heads"], m["dim"], m["vdim"]
+        G = m.get("kv_heads", H)
+        if layer["type"] == "attention":
+            n += (H + G) * dk * W + W * H * dv
+        else:
+            n += (2 * G * dk + 2 * H * dv + 2 * H) * W + W * H * dv
+        n += 2 * layer["mlp"]["ff"] * W
+    return n, lambda B: n
+
+
+def run_ramosun(args):
+    """Ramosun beside Sofopel, the package's closest model (parallel blocks, window attention on the same kernels, a recurrent mixer, the
+    same Linears), at equal width and depth."""
+    from oracle import ramosun_oracle as RO
+    from oracle import sofopel_oracle as SO
+    from llava.model import RamosunConfig, RamosunForCausalLM, SofopelConfig, SofopelForCausalLM
+    from llava._b2 import launch_count
+
+    dev = torch.device("cuda:0")
+    hbm, tfl, src = peaks()
+    pk = {"hbm_gbs": hbm, "bf16_tflops": tfl, "source": src}
+    S, N, layers = args.ctx, 64, 4
+    flush = torch.zeros(160 * 1024 * 1024 // 4, device=dev)  # 160 MB > 126 MB of L2
+    out = {"metric": "Ramosun vs Sofopel (layer-list decoders) at equal width and depth", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+           "peaks": pk, "prompt": S, "decode_steps": N, "l2": "160 MB written before every timed run", "sizes": []}
+    sampler = ClockSampler(0)
+    sampler.start()
+    launches0 = launch_count()
+    for width in [int(w) for w in args.widths.split(",")]:
+        row = {"width": width, "layers": layers}
+        for name, mk_cfg, mk_params, mk_w, cfg_cls, model_cls in (
+                ("ramosun", ramosun_config, ramosun_params, lambda c: RO.random_weights(c, seed=0), RamosunConfig, RamosunForCausalLM),
+                ("sofopel", sofopel_config, sofopel_params, lambda c: SO.random_weights(c, seed=0, ranks={2: 16}), SofopelConfig, SofopelForCausalLM)):
+            cfg = mk_cfg(width, S)
+            w = mk_w(cfg)
+            params, params_read = mk_params(cfg)
+            model = model_cls(cfg_cls(**cfg), {k: torch.from_numpy(np.asarray(v, np.float32)).bfloat16() for k, v in w.items()}, device=dev, dtype=torch.bfloat16,
+                              max_batch=8, max_seq=S + N + 8, max_rows=S)
+            row[name + "_params_total"] = int(sum(v.size for k, v in w.items() if v.ndim == 2 and k != "embed"))
+            del w
+            row[name] = measure_layer_list(model, args, S, N, flush, pk, params, params_read)
+            del model
+        out["sizes"].append(row)
+    out["clocks"] = sampler.stop()
+    out["gpu_launches"] = launch_count() - launches0
+    print(json.dumps(out))
+
+
 def run_katadra(args):
     from oracle import katadra_oracle as KO
     from llava.model import KatadraConfig, KatadraForCausalLM
@@ -1085,10 +1156,11 @@ def run_katadra(args):
 
 def main():
     args = parse_args()
-    if args.arch in ("katadra", "pefivik", "fezuzen", "sofopel"):
+    if args.arch in ("katadra", "pefivik", "fezuzen", "sofopel", "ramosun"):
         if not torch.cuda.is_available():
             raise RuntimeError(f"bench.py --arch {args.arch} needs a B200")
-        return {"katadra": run_katadra, "pefivik": run_pefivik, "fezuzen": run_fezuzen, "sofopel": run_sofopel}[args.arch](args)
+        return {"katadra": run_katadra, "pefivik": run_pefivik, "fezuzen": run_fezuzen, "sofopel": run_sofopel,
+                "ramosun": run_ramosun}[args.arch](args)
     if args.impl == "reference":
         run_reference(args)
     else:
