@@ -125,6 +125,85 @@ __global__ void __launch_bounds__(256) linear_rows_vec_kernel(const float* __res
     }
 }
 
+// ONE row (a decode step of one slot): WPC warps share an output column, each taking every WPC-th run of 256 k, with four 16-byte weight
+// loads per lane in flight; small N gets more warps per column, so that the launch fills the SMs either way. A is read where it lies
+// (it stays in L1), or, when a norm is applied on the way in, staged normed in shared memory while the first weights arrive. The parts of a
+// column meet in shared memory in a fixed order.
+constexpr int R1_U = 4;
+template <typename TW, int WPC, bool NORM>
+__global__ void __launch_bounds__(256) linear_one_row_kernel(const float* __restrict__ A, const TW* __restrict__ W, int64_t ldw,
+                                                             const float* __restrict__ bias, float* __restrict__ out, int N, int K, int act,
+                                                             float alpha, int accumulate, int round_a, DytNorm norm) {
+    extern __shared__ __align__(16) float sA1[];   // [K] with NORM
+    __shared__ float part[8];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int groups = (N + 8 / WPC - 1) / (8 / WPC);   // column groups; with NORM a CTA walks several, so that a row is normed once per CTA
+    constexpr int STEP = WPC * 256;
+    const int kb = ((warp % WPC) * 32 + lane) * 8;
+    float wv[R1_U][8];
+    auto load = [&](int grp, int k0) {
+        const int n = min(grp * (8 / WPC) + warp / WPC, N - 1);   // columns past N read the last row: their sums are never stored
+        const TW* w = W + (size_t)n * ldw;
+#pragma unroll
+        for (int u = 0; u < R1_U; ++u)
+            if (k0 + u * STEP < K) ld_w8(w + k0 + u * STEP, wv[u]);
+    };
+    load(blockIdx.x, kb);
+    if (NORM) {
+        const float al = norm.alpha[0];
+        for (int k = threadIdx.x * 4; k < K; k += 1024) {
+            float4 v = *reinterpret_cast<const float4*>(A + k);
+            const float4 g = *reinterpret_cast<const float4*>(norm.w + k), b = *reinterpret_cast<const float4*>(norm.b + k);
+            v.x = fmaf(tanhf(al * v.x), g.x, b.x); v.y = fmaf(tanhf(al * v.y), g.y, b.y);
+            v.z = fmaf(tanhf(al * v.z), g.z, b.z); v.w = fmaf(tanhf(al * v.w), g.w, b.w);
+            if (round_a) { v.x = round_bf16(v.x); v.y = round_bf16(v.y); v.z = round_bf16(v.z); v.w = round_bf16(v.w); }
+            *reinterpret_cast<float4*>(sA1 + k) = v;
+        }
+        __syncthreads();
+    }
+    for (int grp = blockIdx.x; grp < groups; grp += gridDim.x) {
+        const int n = grp * (8 / WPC) + warp / WPC;
+        float acc = 0.f;
+        for (int k0 = kb; k0 < K; k0 += R1_U * STEP) {
+            if (k0 != kb || grp != blockIdx.x) load(grp, k0);
+#pragma unroll
+            for (int u = 0; u < R1_U; ++u) {
+                const int k = k0 + u * STEP;
+                if (k < K) {
+                    float av[8];
+                    ld_w8((NORM ? sA1 : A) + k, av);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) acc = fmaf(!NORM && round_a ? round_bf16(av[e]) : av[e], wv[u][e], acc);
+                }
+            }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+        if (WPC > 1) {
+            __syncthreads();   // the previous group's parts have been read
+            if (lane == 0) part[warp] = acc;
+            __syncthreads();
+            acc = 0.f;
+#pragma unroll
+            for (int i = 0; i < WPC; ++i) acc += part[(warp / WPC) * WPC + i];
+        }
+        if (lane == 0 && warp % WPC == 0 && n < N) lin_store(out + n, acc, bias, n, act, alpha, accumulate);
+    }
+}
+
+template <typename TW, int WPC>
+int launch_one_row(const LinearArgs& a, cudaStream_t st) {
+    const TW* W = reinterpret_cast<const TW*>(a.W);
+    const int grid = (a.N + 8 / WPC - 1) / (8 / WPC);
+    if (a.norm.alpha != nullptr)
+        linear_one_row_kernel<TW, WPC, true><<<std::min(grid, 4 * num_sms()), 256, (size_t)a.K * sizeof(float), st>>>(a.A, W, a.ldw, a.bias, a.out, a.N, a.K, a.act, a.alpha, a.accumulate,
+                                                                                          a.round_a, a.norm);
+    else
+        linear_one_row_kernel<TW, WPC, false><<<grid, 256, 0, st>>>(a.A, W, a.ldw, a.bias, a.out, a.N, a.K, a.act, a.alpha, a.accumulate, a.round_a, a.norm);
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
 // any K and alignment: one warp per output column, scalar loads
 template <typename TW>
 __global__ void __launch_bounds__(256) linear_rows_kernel(const float* __restrict__ A, int64_t lda, const TW* __restrict__ W, int64_t ldw,
@@ -218,6 +297,14 @@ int launch_linear(const LinearArgs& a, cudaStream_t st) {
     if (a.M <= MR) {
         const bool vec = a.K % 8 == 0 && a.lda % 4 == 0 && a.ldw % 8 == 0 && (reinterpret_cast<uintptr_t>(a.A) & 15) == 0 &&
                          (reinterpret_cast<uintptr_t>(a.W) & 15) == 0;
+        // (with a norm the staged row must fit the default shared-memory limit)
+        if (vec && a.M == 1 && (a.norm.alpha == nullptr || a.K <= 12000)) {
+            const int want = 32 * num_sms();   // warps that keep the SMs busy
+            if (a.N >= want || a.K < 1024) return launch_one_row<TW, 1>(a, st);
+            if (2 * a.N >= want || a.K < 2048) return launch_one_row<TW, 2>(a, st);
+            if (4 * a.N >= want || a.K < 4096) return launch_one_row<TW, 4>(a, st);
+            return launch_one_row<TW, 8>(a, st);
+        }
         if (vec) {
             static bool attr_set = false;
             if (!attr_set) {

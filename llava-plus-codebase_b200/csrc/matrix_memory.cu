@@ -7,15 +7,15 @@
 // what a token needs besides its vectors (unit norms and k . q of the delta rule, decay and write strength, the running maximum) is made
 // once per tile and head. Both dot products of the delta rule run against the state BEFORE the token: with a = S^T k and b = S^T q,
 //     u = beta (v - g a),   S' = g S + k u^T,   y = g b + u (k . q),
-// so the two sums over a column's eight lanes travel together and only u is on the chain from token to token. State, gates and sums are
-// fp32.
+// so only the sum a over a column's eight lanes is on the chain from token to token; the read-outs' sums b meet once per four tokens. State,
+// gates and sums are fp32.
 #include "common.cuh"
 #include "kernels.h"
 
 namespace b2 {
 namespace {
 
-constexpr int MM_TT = 16, MM_L = 8, MM_WARPS = 4, MM_COLS = MM_WARPS * 32 / MM_L, MM_THREADS = MM_WARPS * 32;
+constexpr int MM_TT = 32, MM_L = 8, MM_WARPS = 4, MM_COLS = MM_WARPS * 32 / MM_L, MM_THREADS = MM_WARPS * 32;
 
 __device__ __forceinline__ float mm_softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float mm_log_sigmoid(float v) { return fminf(v, 0.f) - log1pf(expf(-fabsf(v))); }
@@ -182,47 +182,78 @@ __global__ void __launch_bounds__(MM_THREADS) matrix_memory_kernel(MemoryArgs a)
             m_run = __shfl_sync(0xffffffffu, mt, nt - 1);
         }
         __syncthreads();
-        // the next token's vectors are read one token ahead, so that their latency stays off the chain
-        float kn[KPT], qn[KPT];
-        auto read = [&](int t) {
+        // Tokens go in groups of four: a token's vectors are read one token ahead, and the sums that are not on the chain from token to token
+        // (the read-outs) meet once per group, four tokens' worth folded into one value per lane pair.
+        float kb[2][KPT], qb[2][KPT];
+        auto read = [&](int t, float (&kx)[KPT], float (&qx)[KPT]) {
 #pragma unroll
             for (int i = 0; i < KPT; i += 4) {
                 const int off = t * DKP + (i >> 2) * (4 * MM_L) + l * 4;
                 const float4 x = *reinterpret_cast<const float4*>(k + off), y = *reinterpret_cast<const float4*>(q + off);
-                kn[i] = x.x; kn[i + 1] = x.y; kn[i + 2] = x.z; kn[i + 3] = x.w;
-                qn[i] = y.x; qn[i + 1] = y.y; qn[i + 2] = y.z; qn[i + 3] = y.w;
+                kx[i] = x.x; kx[i + 1] = x.y; kx[i + 2] = x.z; kx[i + 3] = x.w;
+                qx[i] = y.x; qx[i + 1] = y.y; qx[i + 2] = y.z; qx[i + 3] = y.w;
             }
         };
-        read(0);
-        for (int t = 0; t < nt; ++t) {
-            float kk[KPT], qq[KPT];
-#pragma unroll
-            for (int i = 0; i < KPT; ++i) { kk[i] = kn[i]; qq[i] = qn[i]; }
+        // one token: updates S, returns this lane's share of the read-out's sum; u: what the delta rule writes (before 1 / |k|)
+        auto step = [&](int t, const float (&kk)[KPT], const float (&qq)[KPT], float& u) {
             const float4 f0 = sC[2 * t];
             const float vt = v[t * MM_COLS + c];
+            float pb[4] = {0.f, 0.f, 0.f, 0.f};
             if (MODE == MEM_DELTA) {
-                const float4 f1 = sC[2 * t + 1];
-                float pa[4] = {0.f, 0.f, 0.f, 0.f}, pb[4] = {0.f, 0.f, 0.f, 0.f};
+                float pa[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-                for (int i = 0; i < KPT; ++i) { pa[i & 3] = fmaf(S[i], kk[i], pa[i & 3]); pb[i & 3] = fmaf(S[i], qq[i], pb[i & 3]); }
-                if (t + 1 < nt) read(t + 1);
-                const float sa = sum8((pa[0] + pa[1]) + (pa[2] + pa[3])), sb = sum8((pb[0] + pb[1]) + (pb[2] + pb[3]));
-                const float u = f0.y * fmaf(-f0.z, sa, vt), uk = u * f1.x;
+                for (int i = 0; i < KPT; ++i) pa[i & 3] = fmaf(S[i], kk[i], pa[i & 3]);
 #pragma unroll
-                for (int i = 0; i < KPT; ++i) S[i] = fmaf(f0.x, S[i], kk[i] * uk);
-                if (l == 0) sO[t * MM_COLS + c] = fmaf(f0.w, sb, u * f1.y);
+                for (int i = 0; i < KPT; ++i) pb[i & 3] = fmaf(S[i], qq[i], pb[i & 3]);
+                const float sa = sum8((pa[0] + pa[1]) + (pa[2] + pa[3]));
+                u = f0.y * fmaf(-f0.z, sa, vt);
+                const float uk = u * sC[2 * t + 1].x;
+#pragma unroll
+                for (int i = 0; i < KPT; ++i) S[i] = fmaf(kk[i], uk, f0.x * S[i]);
             } else {
-                if (t + 1 < nt) read(t + 1);
                 const float wv = f0.y * vt;
-                float pb[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int i = 0; i < KPT; ++i) {
                     S[i] = fmaf(f0.x, S[i], kk[i] * wv);
                     pb[i & 3] = fmaf(S[i], qq[i], pb[i & 3]);
                 }
-                const float sb = a.q_scale * sum8((pb[0] + pb[1]) + (pb[2] + pb[3]));
-                if (l == 0) sO[t * MM_COLS + c] = col == dv ? fmaxf(fabsf(sb), f0.z) + 1e-6f : sb;
             }
+            return (pb[0] + pb[1]) + (pb[2] + pb[3]);
+        };
+        auto finish = [&](int t, float sum, float u) {   // the whole sum of token t's read-out -> its value
+            const float4 f0 = sC[2 * t];
+            if (MODE == MEM_DELTA) return fmaf(f0.w, sum, u * sC[2 * t + 1].y);
+            const float sb = a.q_scale * sum;
+            return col == dv ? fmaxf(fabsf(sb), f0.z) + 1e-6f : sb;
+        };
+        read(0, kb[0], qb[0]);
+        int t = 0;
+        for (; t + 4 <= nt; t += 4) {
+            float p[4], u[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                if (e < 3 || t + 4 < MM_TT) read(t + e + 1, kb[(e + 1) & 1], qb[(e + 1) & 1]);
+                p[e] = step(t + e, kb[e & 1], qb[e & 1], u[e]);
+            }
+            // eight lanes x four sums: lanes with bit 2 set keep tokens 2 and 3, then bit 1 picks one of the two, bit 0 only adds
+            const bool hi = (l & 4) != 0, odd = (l & 2) != 0;
+            float k0 = hi ? p[2] : p[0], k1 = hi ? p[3] : p[1];
+            k0 += __shfl_xor_sync(0xffffffffu, hi ? p[0] : p[2], 4);
+            k1 += __shfl_xor_sync(0xffffffffu, hi ? p[1] : p[3], 4);
+            float sum = odd ? k1 : k0;
+            sum += __shfl_xor_sync(0xffffffffu, odd ? k0 : k1, 2);
+            sum += __shfl_xor_sync(0xffffffffu, sum, 1);
+            const int tk = t + (hi ? 2 : 0) + (odd ? 1 : 0);
+            const float uu = hi ? (odd ? u[3] : u[2]) : (odd ? u[1] : u[0]);
+            const float o = finish(tk, sum, uu);
+            if ((l & 1) == 0) sO[tk * MM_COLS + c] = o;
+        }
+        for (; t < nt; ++t) {   // up to three tokens behind the last group
+            float u = 0.f;
+            const float sum = sum8(step(t, kb[0], qb[0], u));
+            if (t + 1 < nt) read(t + 1, kb[0], qb[0]);
+            const float o = finish(t, sum, u);
+            if (l == 0) sO[t * MM_COLS + c] = o;
         }
         __syncthreads();
         for (int e = tid; e < nt * MM_COLS; e += MM_THREADS) {
