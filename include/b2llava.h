@@ -212,7 +212,8 @@ int b2_batch_set_row(b2_model* m, b2_kv* kv, int slot, int active, const b2_samp
  *                      ga_maps == 2 is differential attention: every query and key head holds TWO maps of ga_dim entries
  *                      each ([map 1 | map 2], the convolution and the rotation act on each), both attend over the same
  *                      values, and a head's output is unit_rms(a1 - lambda a2) * (1 - ga_diff) with ONE learned number
- *                      lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + ga_diff for the layer
+ *                      lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + ga_diff for the layer; ga_qkv_bias adds biases to q, k and v in
+ *                      the projection (in front of convolution and norm)
  *   B2_MIXER_GLA       gated linear attention: S <- diag(alpha) S + k v^T, o = S^T q with q = W_q h * dim^(-1/2) and a decay per
  *                      key channel alpha = sigmoid(W_a2 (W_a1 h) + b)^(1 / gl_tau) through a low-rank pair of matrices; per-head
  *                      RMS norm with one weight vector for all heads, SiLU(W_g h) gate, out-projection
@@ -221,7 +222,8 @@ int b2_batch_set_row(b2_model* m, b2_kv* kv, int slot, int active, const b2_samp
  * floor(i / mask_size) == floor(j / mask_size), chunks counted from position 0 of the sequence.
  * Rotation (rot_*): pairs (2m, 2m+1), m < rot_dims / 2, of a head turn by p * f_m, f_m = rot_base^(-2m / rot_dims); with
  * rot_factor > 0 the frequencies are blended towards f_m / rot_factor over the pairs whose wavelength lies between
- * rot_original / rot_fast and rot_original / rot_slow turns (YaRN) and cos / sin carry the factor 0.1 ln(rot_factor) + 1.
+ * rot_original / rot_fast and rot_original / rot_slow turns (YaRN) and cos / sin carry the factor 0.1 ln(rot_factor) + 1
+ * (rot_scaling: B2_ROT_BANDS scales by bands of wavelength instead, B2_ROT_LINEAR divides every f_m by rot_factor).
  * Blocks: B2_BLOCK_POST_LN adds the LayerNorm of every sublayer's OUTPUT; B2_BLOCK_PRE_RMS1 is pre-norm,
  * x += residual_mult * sublayer(g * unit_rms(x)) with ONE learned number g per norm (also in front of the head);
  * B2_BLOCK_SANDWICH_RMS norms both sides with weighted RMS norms, x += rms_w'(sublayer(u + conv(u))), u = rms_w(x), where
@@ -231,12 +233,15 @@ int b2_batch_set_row(b2_model* m, b2_kv* kv, int slot, int active, const b2_samp
  * B2_BLOCK_PARALLEL2: parallel with a norm for each sublayer, x += residual_mult * (mixer(N1(x)) + ff(N2(x))), both norms of the same x. norm_kind of
  * the two parallel blocks: weighted RMS norm, or the dynamic tanh N(x) = tanh(alpha x) w + b (no statistics; alpha one number).
  * Feed-forwards: B2_FF_GELU (W_down gelu(W_up x), the erf form), B2_FF_CLAMP_GLU (W_down (a(g) (u + 1)) with g = min(W_gate x, ff_limit), u = clamp(W_up x, +-ff_limit),
- * a(g) = g sigmoid(ff_act_slope g)), B2_FF_RELU_SQ (W_down relu(W_up x)^2), B2_FF_POLYNORM (biased projections around
+ * a(g) = g sigmoid(ff_act_slope g)), B2_FF_GELU_GLU (W_down (gelu(W_gate x) * (W_up x)), the tanh form), B2_FF_RELU_SQ (W_down relu(W_up x)^2), B2_FF_POLYNORM (biased projections around
  * a N(z) + b N(z^2) + c N(z^3) + e, N = division by the token's root mean square), B2_FF_MOE (router, group-limited
  * top-k, experts without biases, optional shared expert; moe_score: sigmoid or softmax scores; moe_group_score: a group counts
  * by its two best experts or by its best; moe_raw_weights: the chosen scores are the weights as they are, else divided by their
- * sum and scaled; moe_act: SiLU-gated experts or W_down relu(W_up x)^2).
- * A model may add a hashed bigram row to every token embedding, loop a block of layers several times with the same tensors
+ * sum and scaled; moe_act: SiLU-gated experts, W_down relu(W_up x)^2, or the bounded gated unit of B2_FF_CLAMP_GLU with ff_limit and
+ * ff_act_slope; moe_correction: a learned number per expert joins the scores for the choice of groups and experts only; moe_identity:
+ * that many further rows of the router, behind the experts, are identity experts: chosen like experts (groups span both), no tensors,
+ * their output is the sublayer's input).
+ * A model may norm its token embeddings (embed_norm: weighted RMS norm, tensor embed.norm), add a hashed bigram row to every token embedding, loop a block of layers several times with the same tensors
  * (every pass has its own cache/state; before a pass the embedding output is added again from the second pass on, and a
  * learned per-pass vector always; loop_plain: nothing is added between the passes; loop_mix: x becomes W_in [x; embedding output] in front
  * of every pass), scale its token embedding, use the embedding table as its head, and soft-cap its logits with tanh.
@@ -248,17 +253,17 @@ int b2_batch_set_row(b2_model* m, b2_kv* kv, int slot, int active, const b2_samp
 enum { B2_ARCH_LLAVA = 0, B2_ARCH_LAYER_LIST = 1 };
 enum { B2_MIXER_MAMBA2 = 1, B2_MIXER_PARALLEL = 2, B2_MIXER_LATENT_ATTN = 3, B2_MIXER_HGRN2 = 4, B2_MIXER_GQA_ATTN = 5, B2_MIXER_GLA = 6, B2_MIXER_MLSTM = 7,
        B2_MIXER_DELTA = 8 };
-enum { B2_FF_RELU_SQ = 0, B2_FF_POLYNORM = 1, B2_FF_MOE = 2, B2_FF_CLAMP_GLU = 3, B2_FF_GELU = 4 };
+enum { B2_FF_RELU_SQ = 0, B2_FF_POLYNORM = 1, B2_FF_MOE = 2, B2_FF_CLAMP_GLU = 3, B2_FF_GELU = 4, B2_FF_GELU_GLU = 5 };
 enum { B2_BLOCK_POST_LN = 0, B2_BLOCK_PRE_RMS1 = 1, B2_BLOCK_SANDWICH_RMS = 2, B2_BLOCK_PARALLEL_RMS = 3, B2_BLOCK_PARALLEL2 = 4 };
 enum { B2_NORM_RMS = 0, B2_NORM_DYT = 1 };
 enum { B2_QK_NORM_NONE = 0, B2_QK_NORM_HEAD = 1, B2_QK_NORM_ALL = 2 };
 enum { B2_SINK_NONE = 0, B2_SINK_FIXED = 1, B2_SINK_HEAD = 2 };
-enum { B2_ROT_YARN = 0, B2_ROT_BANDS = 1 };
+enum { B2_ROT_YARN = 0, B2_ROT_BANDS = 1, B2_ROT_LINEAR = 2 };
 enum { B2_GATE_CHANNEL = 0, B2_GATE_HEAD = 1, B2_GATE_NONE = 2 };
 enum { B2_MASK_CAUSAL = 0, B2_MASK_WINDOW = 1, B2_MASK_CHUNK = 2 };
 enum { B2_MOE_SCORE_SIGMOID = 0, B2_MOE_SCORE_SOFTMAX = 1 };
 enum { B2_MOE_GROUP_TOP2_SUM = 0, B2_MOE_GROUP_MAX = 1 };
-enum { B2_MOE_ACT_SWIGLU = 0, B2_MOE_ACT_RELU_SQ = 1 };
+enum { B2_MOE_ACT_SWIGLU = 0, B2_MOE_ACT_RELU_SQ = 1, B2_MOE_ACT_CLAMP_GLU = 2 };
 enum { B2_COMPUTE_BF16 = 0, B2_COMPUTE_F32 = 1 };
 typedef struct b2_seq_layer_desc {
     int32_t type;            /* B2_MIXER_* */
@@ -316,6 +321,9 @@ typedef struct b2_seq_layer_desc {
     float ml_cap;
     /* B2_MIXER_DELTA: gated delta rule behind a convolution of dn_conv taps with SiLU on q, k, v; dn_kv_heads query / key heads */
     int32_t dn_heads, dn_kv_heads, dn_dim, dn_vdim, dn_conv;
+    int32_t ga_qkv_bias;     /* B2_MIXER_GQA_ATTN: biases on q, k and v (mix.q.b, mix.k.b, mix.v.b) */
+    /* B2_FF_MOE: corrected choice scores (mlp.correction), identity experts behind the moe_experts (rows of mlp.router and of the correction) */
+    int32_t moe_correction, moe_identity;
 } b2_seq_layer_desc;
 typedef struct b2_seq_model_desc {
     int32_t width, vocab, n_layers;
@@ -336,6 +344,7 @@ typedef struct b2_seq_model_desc {
     int32_t norm_kind;       /* B2_NORM_*, of B2_BLOCK_PARALLEL_RMS / PARALLEL2 */
     int32_t tied_head;       /* logits = embed N(x): no head tensor */
     int32_t loop_mix;        /* parallel blocks: x <- W_in [x; x0] in front of every pass, x0 the embedding output (tensor loop.in; no loop.step) */
+    int32_t embed_norm;      /* x = rms_w(embed[token]) with tensor embed.norm; not with bigram rows, embed_scale or a kept embedding output */
 } b2_seq_model_desc;
 int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* layers, b2_model** out);
 /* Layer RUNS of one forward pass (a looped layer counts every time): rows of b2_append_tokens' resid_out; -1 for other models */
@@ -350,8 +359,8 @@ int b2_seq_model_runs(const b2_model* m);
  * ([width, taps]), l<i>.mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,o} (latent attention; no dkv* with la_kv_from),
  * l<i>.mix.{q,k,v,q.conv,k.conv,v.conv,g,o} (grouped attention), l<i>.mlp.{router,e<j>.up,e<j>.down,shared.up,shared.down}.
  * B2_BLOCK_PARALLEL_RMS models: embed, head, final.norm, l<i>.norm1 (width each), l<i>.mix.{q,k,v,o} with, by the layer's options,
- * {q,k,v}.conv, {q,k}.norm, g, {lq1,lk1,lq2,lk2} (grouped attention), l<i>.mix.{q,k,v,g,a1,a2,a2.b,norm,o} (gated linear attention),
- * l<i>.mlp.{gate,up,down}.
+ * {q,k,v}.b, {q,k,v}.conv, {q,k}.norm, g, {lq1,lk1,lq2,lk2} (grouped attention), l<i>.mix.{q,k,v,g,a1,a2,a2.b,norm,o} (gated linear attention),
+ * l<i>.mlp.{gate,up,down}; embed_norm: embed.norm; experts also l<i>.mlp.correction.
  * B2_BLOCK_PARALLEL2 models: the same with l<i>.norm2; with norm_kind DYT every norm also has .b (width) and .alpha (one number); tied_head: no
  * head; loop_mix: loop.in [width, 2 width] (x's columns first); l<i>.mix.{q,k,v,g,i,i.b,f,f.b,norm,o} (mLSTM),
  * l<i>.mix.{q,k,v,q.conv,k.conv,v.conv,b,a,A_log,dt_bias,g,norm,o} (delta rule), mix.sink (grouped attention with B2_SINK_HEAD). */

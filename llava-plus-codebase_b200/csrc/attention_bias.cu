@@ -38,6 +38,14 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// the last write of one output entry: its own sigmoid gate, when there is one, and the form the output is wanted in
+__device__ __forceinline__ void store_out(const BiasAttnArgs& a, int row, int head, int d, float v) {
+    if (a.chan_gate != nullptr) v /= 1.f + expf(-a.chan_gate[(size_t)row * a.ldg + (size_t)head * a.dv + d]);
+    const size_t at = (size_t)row * a.ldo + (size_t)head * a.dv + d;
+    if (a.out16 != nullptr) reinterpret_cast<__nv_bfloat16*>(a.out16)[at] = __float2bfloat16_rn(v);
+    else a.out[at] = v;
+}
+
 // unit = q head (normalise, temperature, in place) | k head (normalise, append) | v head (append)
 __global__ void attn_prepare_kernel(BiasAttnArgs a) {
     const int units = a.H + 2 * a.G;
@@ -160,7 +168,7 @@ __global__ void __launch_bounds__(AT_WARPS * 32) attn_bias_kernel(BiasAttnArgs a
 #pragma unroll
         for (int c = 0; c < AT_MAXC; ++c) {
             const int d = lane + 32 * c;
-            if (d < a.dv) a.out[(size_t)r * a.ldo + (size_t)h * a.dv + d] = o[c] * inv;
+            if (d < a.dv) store_out(a, r, h, d, o[c] * inv);
         }
     }
 }
@@ -369,7 +377,7 @@ __global__ void __launch_bounds__(TL_WARPS * 32, MAXC == 16 ? 1 : 2) attn_tile_k
 #pragma unroll
             for (int c = 0; c < MAXC; ++c) {
                 const int d = lane + 32 * c;
-                if (d < dv) a.out[(size_t)row * a.ldo + (size_t)head * dv + d] = o[i][c] * inv;
+                if (d < dv) store_out(a, row, head, d, o[i][c] * inv);
             }
         }
     }
@@ -416,7 +424,7 @@ __global__ void __launch_bounds__(512) attn_merge_kernel(BiasAttnArgs a) {
             acc = fmaf(p0, wgt[s], acc); acc = fmaf(p1, wgt[s + 1], acc); acc = fmaf(p2, wgt[s + 2], acc); acc = fmaf(p3, wgt[s + 3], acc);
         }
         for (; s < a.nsplit; ++s) acc = fmaf(part[(size_t)s * stride + 2 + d], wgt[s], acc);
-        a.out[(size_t)r * a.ldo + (size_t)h * a.dv + d] = acc * inv;
+        store_out(a, r, h, d, acc * inv);
     }
 }
 
@@ -456,7 +464,7 @@ int launch_tile(const BiasAttnArgs& a, int QT, int HC, dim3 grid, size_t smem, c
 
 int attn_bias_f32(const BiasAttnArgs& a, cudaStream_t st) {
     B2_TRY(check_args(a, "attn_bias"));
-    B2_CHECK_ARG(a.out && (a.rel == nullptr || a.bucket_of != nullptr), "attn_bias: null argument");
+    B2_CHECK_ARG((a.out || a.out16) && (a.rel == nullptr || a.bucket_of != nullptr), "attn_bias: null argument");
     B2_CHECK_ARG(a.nsplit >= 1 && a.nsplit <= 64 && (a.nsplit == 1 || a.partial != nullptr), "attn_bias: 1..64 key splits, with scratch");
     const int warps = a.rows * a.H;
     const bool vec = a.dk % 4 == 0 && (reinterpret_cast<uintptr_t>(a.kcache) & 15) == 0;

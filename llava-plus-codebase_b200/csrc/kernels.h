@@ -294,6 +294,17 @@ int linear_f32(const LinearArgs& a, cudaStream_t stream);
 // out[r, :K] = bf16(A[r, :K]): the A operand of a tensor-core GEMM from fp32 activations (ld_out % 8 == 0)
 int cast_rows_bf16(const float* A, int64_t lda, void* out, int64_t ld_out, int M, int K, cudaStream_t stream);
 
+// The gated unit in its general form: with g = in[r, c] and u = in[r, ff + c], limit > 0 first bounds them, g = min(g, limit),
+// u = clamp(u, -limit, limit); out = a(g) (u + up_shift) with a(g) = g sigmoid(slope g), or (GLU_GELU_TANH) the tanh form of GELU,
+// a(g) = g / 2 (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))). (slope 1, no limit, shift 0: SiLU(g) u.)
+enum { GLU_SIGMOID = 0, GLU_GELU_TANH = 1 };
+struct GluAct { float slope = 1.f, limit = 0.f, up_shift = 0.f; int kind = GLU_SIGMOID; };
+__host__ __device__ inline float glu_act(float g, float u, const GluAct& a) {
+    if (a.limit > 0.f) { g = fminf(g, a.limit); u = fminf(fmaxf(u, -a.limit), a.limit); }
+    const float v = a.kind == GLU_GELU_TANH ? 0.5f * g * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * g * g, g, g))) : g / (1.f + expf(-a.slope * g));
+    return v * (u + a.up_shift);
+}
+
 // Grouped Linear: output rows come in tiles of tile_rows (1 or 64) rows; tile t multiplies with the weight matrix of group
 // tile_group[t] (W + group * w_group_stride elements; a negative group: the tile is unused). Output row m reads input row
 // a_rows[m] (a_rows null: m / a_div; negative: a zero row). out[m, :N] = act(A[src] W_g^T); M bounds the rows (the launch grid).
@@ -307,9 +318,22 @@ struct GroupedLinearArgs {
     int act = LIN_NONE;
     int round_a = 0;
     int swiglu = 0;   // one-row tiles only: a group's matrix is [gate | up] of N rows each and out[m, n] = silu(gate_n . a) * (up_n . a)
-    float glu_slope = 1.f, glu_limit = 0.f, glu_up_shift = 0.f;   // with swiglu: the general gated unit (GluAct) instead of SiLU(g) u
+    GluAct glu;       // with swiglu: the gated unit (default: SiLU(g) u)
 };
 int linear_grouped_f32(const GroupedLinearArgs& g, cudaStream_t stream);
+// The second products of a handful of tokens' experts and their weighted sum in one launch (a decode step): with e_k = idx[r, k] < E,
+// x[r, n] += alpha * sum_k w[r, k] * (W[e_k * w_group_stride + n * K ..] . a[r * top + k]); e_k < 0: an identity expert, which adds
+// w[r, k] * h[r, n]. W has N rows of K entries per expert.
+struct ExpertSumArgs {
+    const float* a = nullptr; int64_t lda = 0;   // fp32 [rows * top, K]
+    const void* W = nullptr; int64_t w_group_stride = 0; int w_dtype = DT_F32;
+    const int32_t* idx = nullptr; const float* w = nullptr;
+    const float* h = nullptr; int64_t ldh = 0;   // identity experts' input (may be null when no index is negative)
+    float* x = nullptr; int64_t ldx = 0;
+    int rows = 0, top = 0, N = 0, K = 0, round_a = 0;
+    float alpha = 1.f;
+};
+int expert_sum_f32(const ExpertSumArgs& a, cudaStream_t stream);
 // `batch` small Linears in one launch on a handful of rows (a decode step's per-head products): for b < batch,
 // out[m, b * o_bs + n] = sum_k A[m, b * a_bs + k] * W[b * w_bs + n * K + k], m < M <= 8; weights in w_dtype, fp32 accumulation;
 // gate (nullable, [M, ldg]): the result is multiplied by sigmoid(gate[m, b])
@@ -321,39 +345,34 @@ enum { GROUPED_TILE_ROWS = 64 };
 // Router: scores s = sigmoid(logits) (score_fn MOE_SCORE_SOFTMAX: softmax over the experts); experts form `groups` equal groups of
 // neighbours, a group's score is the sum of its two largest scores (group_score MOE_GROUP_MAX: its largest), only experts of
 // the best `keep` groups compete; the `top` largest are chosen (ties: the lower index); w = s / (sum of the chosen s + 1e-20) *
-// scale (raw_weights: w = s). idx / w: [rows, top].
+// scale (raw_weights: w = s). correction (nullable, [experts]): groups and experts are compared by s + correction, the weights use
+// s alone. The last `identity` of the experts hand their input on: they compete as the others do and get index -1. idx / w: [rows, top].
 enum { MOE_SCORE_SIGMOID = 0, MOE_SCORE_SOFTMAX = 1, MOE_GROUP_TOP2_SUM = 0, MOE_GROUP_MAX = 1 };   // the values of B2_MOE_*
 struct MoeRouteArgs {
     const float* logits = nullptr; int64_t ld = 0;
     int rows = 0, experts = 0, top = 0, groups = 1, keep = 1;
     int score_fn = 0, group_score = 0, raw_weights = 0;
+    int identity = 0;
+    const float* correction = nullptr;
     float scale = 1.f;
     int32_t* idx = nullptr; float* w = nullptr;
 };
 int moe_route_f32(const MoeRouteArgs& a, cudaStream_t stream);
-// Sorts the rows * top pairs by expert into tiles of `tile` rows of one expert each: pair_pos[pair] = its position,
+// Sorts the rows * top pairs by expert into tiles of `tile` rows of one expert each: pair_pos[pair] = its position (-1: a pair without
+// expert, idx < 0, has none),
 // src_row[position] = its token row (-1: padding), tile_group[t] = the expert of tile t (-1: unused).
 // max_tiles * tile >= rows * top + experts * (tile - 1).
 int moe_plan(const int32_t* idx, int rows, int top, int experts, int tile, int max_tiles, int32_t* pair_pos, int32_t* src_row, int32_t* tile_group,
              cudaStream_t stream);
-// out[r, c] = silu(in[r, c]) * in[r, ff + c], c < ff; out16 (nullable, bf16 [rows, ld_out16]) receives the rounded copy that a
+// out[r, c] = glu_act(in[r, c], in[r, ff + c]), c < ff; out16 (nullable, bf16 [rows, ld_out16]) receives the rounded copy that a
 // tensor-core product reads next (out may then be null)
-int swiglu_rows_f32(const float* in, int64_t ld_in, float* out, int64_t ld_out, int rows, int ff, cudaStream_t stream, void* out16 = nullptr,
-                    int64_t ld_out16 = 0);
-// The gated unit in its general form: with g = in[r, c] and u = in[r, ff + c], limit > 0 first bounds them, g = min(g, limit),
-// u = clamp(u, -limit, limit); out = g sigmoid(slope g) (u + up_shift). (slope 1, no limit, shift 0: SiLU(g) u.)
-struct GluAct { float slope = 1.f, limit = 0.f, up_shift = 0.f; };
-__host__ __device__ inline float glu_act(float g, float u, const GluAct& a) {
-    if (a.limit > 0.f) { g = fminf(g, a.limit); u = fminf(fmaxf(u, -a.limit), a.limit); }
-    return g / (1.f + expf(-a.slope * g)) * (u + a.up_shift);
-}
 int glu_rows_f32(const float* in, int64_t ld_in, float* out, int64_t ld_out, int rows, int ff, const GluAct& act, cudaStream_t stream,
                  void* out16 = nullptr, int64_t ld_out16 = 0);
 // out[p, :K] = bf16(A[src_row[p], :K]), zeros where src_row[p] < 0: the gathered A operand of a grouped tensor-core product
 int gather_rows_bf16(const float* A, int64_t lda, const int32_t* src_row, void* out, int64_t ld_out, int rows, int K, cudaStream_t stream);
-// x[r] += alpha * sum_k w[r, k] * y[pair_pos[r * top + k]] (pair_pos null: the pair's own index)
+// x[r] += alpha * sum_k w[r, k] * y[pair_pos[r * top + k]] (a negative position: an identity expert, h[r] in y's place)
 int moe_combine_f32(float* x, const float* y, int64_t ldy, const int32_t* pair_pos, const float* w, int rows, int top, int cols, float alpha,
-                    cudaStream_t stream);
+                    cudaStream_t stream, const float* h = nullptr, int64_t ldh = 0);
 
 // ---- fp32 norms and row helpers (norms_f32.cu) ------------------------------------------------------------------------
 // x[r] += LayerNorm(y[r]) * gamma + beta   (normalisation of a sublayer's OUTPUT, added to the residual stream)
@@ -397,7 +416,8 @@ int latent_append_f32(const float* in, int64_t ld_in, const float* gamma, float*
                       int rank, int Smax, float eps, cudaStream_t stream);
 // x[r, :] = table[tokens[r], :] as fp32; ids outside [0, vocab) give a zero row and raise *err_flag (B2_ERR_TOKEN_RANGE)
 int embed_rows_f32(const int32_t* tokens, const void* table, int table_dtype, float* x, int rows, int cols, int vocab, int* err_flag,
-                   cudaStream_t stream, float scale = 1.f);   // scale: x = table[token] * scale, in fp32
+                   cudaStream_t stream, float scale = 1.f,    // scale: x = table[token] * scale, in fp32
+                   const float* norm_w = nullptr, float eps = 0.f);   // norm_w (not with scale): the row is divided by sqrt(mean(x^2) + eps) and weighted
 // Differential attention, per (row, head): d = a1 - lambda a2 over the head's dv values, out = d / sqrt(mean(d^2) + eps) * out_scale.
 // y holds map 1 of every head, then map 2 of every head: [rows, 2 * heads * dv]
 int diff_combine_f32(const float* y, int64_t ldy, float* out, int64_t ldo, int rows, int heads, int dv, float lambda, float out_scale, float eps,
@@ -406,9 +426,9 @@ int diff_combine_f32(const float* y, int64_t ldy, float* out, int64_t ldo, int r
 int sigmoid_gate_f32(const float* a, int64_t lda, const float* g, int64_t ldg, float* out, int64_t ldo, int rows, int cols, cudaStream_t stream);
 
 // out[i] = x[row_index[i]] / sqrt(mean(x^2) + eps) * w (row_index null: row i; rows of pitch ld_in / ld_out); accumulate: out[i] += ...
-// (a normed sublayer output joining the residual stream)
+// (a normed sublayer output joining the residual stream); out16 (nullable, bf16 [rows, cols], not with accumulate): a rounded copy as well
 int rms_weight_f32(const float* in, int64_t ld_in, const int32_t* row_index, const float* w, float* out, int64_t ld_out, int accumulate, int rows,
-                   int cols, float eps, cudaStream_t stream);
+                   int cols, float eps, cudaStream_t stream, void* out16 = nullptr);
 
 // One or two dynamic-tanh norms of the same (gathered) rows in one pass: row r of an output is N(x[row_index[r]]) (row_index null: row r),
 // as fp32 (out, pitch cols) or as the bf16 operand of a tensor-core product (out16, pitch cols).
@@ -438,7 +458,8 @@ int sandwich_norm_f32(const SandwichNormArgs& a, cudaStream_t stream);
 // (2 ln base), and cos / sin are scaled by 0.1 ln(factor) + 1.
 // factor > 0, scaling ROT_BANDS: f_m stays where its wavelength l = 2 pi / f_m is below original / fast, becomes f_m / factor above original / slow,
 // and (1 - s) f_m / factor + s f_m, s = (original / l - slow) / (fast - slow), in between; cos / sin are not scaled.
-enum { ROT_YARN = 0, ROT_BANDS = 1 };   // the values of B2_ROT_*
+// factor > 0, scaling ROT_LINEAR: every f_m becomes f_m / factor.
+enum { ROT_YARN = 0, ROT_BANDS = 1, ROT_LINEAR = 2 };   // the values of B2_ROT_*
 struct RotaryDesc { int dims = 0; float base = 10000.f, factor = 0.f, original = 0.f, fast = 0.f, slow = 0.f; int scaling = ROT_YARN; };
 // table_dev[p][m] = (cos, sin)(p * f_m) * scale for p < positions; computed on the host in double precision
 int rotary_table_build(const RotaryDesc& d, int positions, float2* table_dev);
@@ -559,6 +580,8 @@ struct BiasAttnArgs {
     int Gv = 0;                                   // > 0: vcache holds Gv <= G value heads per slot and key head g reads value head g mod Gv
                                                   // (the maps of differential attention: G = maps * Gv key heads over one set of values)
     const float* head_gate = nullptr; int64_t ldg = 0;   // non-null ([rows, ldg], entry h): a head's output is multiplied by sigmoid(head_gate[r, h])
+    const float* chan_gate = nullptr;             // non-null ([rows, ldg], entry h * dv + d): every entry of the output has a sigmoid gate of its own
+    void* out16 = nullptr;                        // non-null: the output is written as bf16 (pitch ldo) instead of fp32: the operand of a product
     float* partial = nullptr; int nsplit = 1;     // split-KV scratch [rows*H*nsplit*(dv+2)] when nsplit > 1
     int tile_rows = 0;                            // consecutive rows that share a slot (a prompt portion: its rows; a decode step: 1);
                                                   // 0: one warp per (row, head) without shared key/value tiles

@@ -440,9 +440,66 @@ __global__ void __launch_bounds__(256) linear_grouped_rows_kernel(GroupedLinearA
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) { acc += __shfl_xor_sync(0xffffffffu, acc, o); acc2 += __shfl_xor_sync(0xffffffffu, acc2, o); }
     if (lane == 0) {
-        if (g.swiglu) g.out[(size_t)m * g.ld_out + n] = glu_act(acc, acc2, GluAct{g.glu_slope, g.glu_limit, g.glu_up_shift});   // silu(gate) * up, or its bounded form
+        if (g.swiglu) g.out[(size_t)m * g.ld_out + n] = glu_act(acc, acc2, g.glu);   // silu(gate) * up, or its bounded form
         else lin_store(g.out + (size_t)m * g.ld_out + n, acc, nullptr, n, g.act, 1.f, 0);
     }
+}
+
+// A decode step's second expert products with the weighted sum over a token's choices: one warp per (token, output column) walks the
+// choices in their order and adds the finished sum onto x, so that no per-pair output is written and read back. VEC: a lane keeps up to
+// four weight loads of 16 bytes in flight per choice.
+template <typename TW, bool VEC>
+__global__ void __launch_bounds__(256) expert_sum_kernel(ExpertSumArgs a) {
+    const int r = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int n = blockIdx.x * 8 + warp;
+    if (n >= a.N) return;
+    float total = 0.f;
+    for (int c = 0; c < a.top; ++c) {
+        const int p = r * a.top + c, e = a.idx[p];
+        float y;
+        if (e < 0) {
+            y = a.h[(size_t)r * a.ldh + n];
+        } else {
+            const TW* w = reinterpret_cast<const TW*>(a.W) + (size_t)e * a.w_group_stride + (size_t)n * a.K;
+            const float* v = a.a + (size_t)p * a.lda;
+            float acc = 0.f;
+            if (VEC) {
+                for (int k0 = lane * 8; k0 < a.K; k0 += 1024) {
+                    float wv[4][8];
+#pragma unroll
+                    for (int u = 0; u < 4; ++u)
+                        if (k0 + u * 256 < a.K) ld_w8(w + k0 + u * 256, wv[u]);
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        if (k0 + u * 256 < a.K) {
+                            float av[8];
+                            ld_w8(v + k0 + u * 256, av);
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) acc = fmaf(a.round_a ? round_bf16(av[i]) : av[i], wv[u][i], acc);
+                        }
+                    }
+                }
+            } else {
+                for (int k = lane; k < a.K; k += 32) acc = fmaf(a.round_a ? round_bf16(v[k]) : v[k], ld_w(w + k), acc);
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+            y = acc;
+        }
+        total = fmaf(a.w[p], y, total);
+    }
+    if (lane == 0) a.x[(size_t)r * a.ldx + n] += a.alpha * total;
+}
+
+template <typename TW>
+int launch_expert_sum(const ExpertSumArgs& a, cudaStream_t st) {
+    const bool vec = a.K % 8 == 0 && a.lda % 4 == 0 && a.w_group_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(a.a) & 15) == 0 &&
+                     (reinterpret_cast<uintptr_t>(a.W) & 15) == 0;
+    dim3 grid((a.N + 7) / 8, a.rows);
+    if (vec) expert_sum_kernel<TW, true><<<grid, 256, 0, st>>>(a);
+    else expert_sum_kernel<TW, false><<<grid, 256, 0, st>>>(a);
+    B2_LAUNCH_CHECK();
+    return 0;
 }
 
 // batched small Linears of a decode step: block = 8 output columns of one batch entry (a head), one warp per column; the
@@ -536,6 +593,12 @@ int linear_grouped_f32(const GroupedLinearArgs& g, cudaStream_t st) {
     B2_CHECK_ARG(g.a_rows != nullptr || g.a_div >= 1, "linear_grouped: no source rows");
     B2_CHECK_ARG(g.w_dtype == DT_F32 || g.w_dtype == DT_BF16, "linear_grouped: weights must be fp32 or bf16");
     return g.w_dtype == DT_F32 ? launch_grouped<float>(g, st) : launch_grouped<__nv_bfloat16>(g, st);
+}
+
+int expert_sum_f32(const ExpertSumArgs& a, cudaStream_t st) {
+    B2_CHECK_ARG(a.a && a.W && a.idx && a.w && a.x && a.rows > 0 && a.top > 0 && a.N > 0 && a.K > 0, "expert_sum: bad argument");
+    B2_CHECK_ARG(a.w_dtype == DT_F32 || a.w_dtype == DT_BF16, "expert_sum: weights must be fp32 or bf16");
+    return a.w_dtype == DT_F32 ? launch_expert_sum<float>(a, st) : launch_expert_sum<__nv_bfloat16>(a, st);
 }
 
 namespace {

@@ -1,4 +1,5 @@
-// Mixture-of-experts feed-forward of the layer-list decoders: sigmoid or softmax router with group-limited top-k choice, the plan that
+// Mixture-of-experts feed-forward of the layer-list decoders: sigmoid or softmax router with group-limited top-k choice, optionally by
+// corrected scores and with identity experts (index -1: the token's input itself is the output), the plan that
 // sorts (token, choice) pairs by expert into tiles of one expert each, the gated activation, and the weighted sum of the
 // chosen experts' outputs. The expert products themselves are grouped Linears (linear_generic.cu). Router scores, the choice
 // and the weights are fp32; the order of a pair inside its expert's tile does not change its result, and the sum over a
@@ -21,16 +22,17 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
     }
 }
 
-// One warp per row. Shared memory per warp: E scores, G group scores (later: group alive flags), E taken flags.
+// One warp per row. Shared memory per warp: E scores, G group scores (later: group alive flags), E taken flags, E choice scores.
 __global__ void moe_route_kernel(MoeRouteArgs a) {
     extern __shared__ float sm[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = blockIdx.x * (blockDim.x >> 5) + warp;
     if (r >= a.rows) return;
     const int E = a.experts, G = a.groups, per = E / G;
-    float* s = sm + (size_t)warp * (2 * E + G);
+    float* s = sm + (size_t)warp * (3 * E + G);
     float* gs = s + E;
     float* taken = gs + G;
+    float* c = taken + E;   // what is compared: the score, or the score plus its correction (it may be negative)
     if (a.score_fn == MOE_SCORE_SOFTMAX) {
         float mx = -INFINITY;
         for (int e = lane; e < E; e += 32) mx = fmaxf(mx, a.logits[(size_t)r * a.ld + e]);
@@ -51,12 +53,13 @@ __global__ void moe_route_kernel(MoeRouteArgs a) {
             taken[e] = 0.f;
         }
     }
+    for (int e = lane; e < E; e += 32) c[e] = a.correction != nullptr ? s[e] + a.correction[e] : s[e];   // each lane reads back its own scores
     __syncwarp();
     // a group's score: the sum of its two largest scores (of its one score, when a group is a single expert), or its largest
     for (int g = lane; g < G; g += 32) {
         float b1 = -INFINITY, b2v = -INFINITY;
         for (int e = g * per; e < (g + 1) * per; ++e) {
-            const float v = s[e];
+            const float v = c[e];
             if (v > b1) { b2v = b1; b1 = v; } else if (v > b2v) { b2v = v; }
         }
         gs[g] = (per > 1 && a.group_score != MOE_GROUP_MAX) ? b1 + b2v : b1;
@@ -81,23 +84,25 @@ __global__ void moe_route_kernel(MoeRouteArgs a) {
         float bv = -INFINITY;
         int bi = -1;
         for (int e = lane; e < E; e += 32)
-            if (taken[e] == 0.f && (bi < 0 || s[e] > bv)) { bv = s[e]; bi = e; }
+            if (taken[e] == 0.f && (bi < 0 || c[e] > bv)) { bv = c[e]; bi = e; }
         warp_argmax(bv, bi);
-        if (bi < 0) { bi = 0; bv = 0.f; }   // fewer candidates than choices: a zero-weight pair on expert 0
+        float sv = 0.f;
+        if (bi < 0) bi = 0;   // fewer candidates than choices: a zero-weight pair on expert 0
+        else sv = s[bi];
         if (lane == 0) taken[bi] = 1.f;
         __syncwarp();
-        if (lane == k) { mine = bv; mine_e = bi; }
-        sum += bv;
+        if (lane == k) { mine = sv; mine_e = bi; }
+        sum += sv;
     }
     if (lane < a.top) {
-        a.idx[(size_t)r * a.top + lane] = mine_e;
+        a.idx[(size_t)r * a.top + lane] = mine_e < E - a.identity ? mine_e : -1;
         a.w[(size_t)r * a.top + lane] = a.raw_weights ? mine : mine / (sum + 1e-20f) * a.scale;
     }
 }
 
 // One block. pairs = rows * top (token, choice) pairs with their expert in idx. Every expert gets its pairs in consecutive
 // positions, padded to a multiple of `tile` rows: pair_pos[pair] = position, src_row[position] = token row (-1: padding),
-// tile_group[t] = expert of tile t (-1: unused), for max_tiles tiles.
+// tile_group[t] = expert of tile t (-1: unused), for max_tiles tiles. A pair with a negative index has no expert: position -1.
 __global__ void __launch_bounds__(1024) moe_plan_kernel(const int32_t* __restrict__ idx, int pairs, int top, int experts, int tile, int max_tiles,
                                                         int32_t* __restrict__ pair_pos, int32_t* __restrict__ src_row,
                                                         int32_t* __restrict__ tile_group) {
@@ -107,7 +112,8 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int32_t* __restric
     for (int p = threadIdx.x; p < max_tiles * tile; p += blockDim.x) src_row[p] = -1;
     for (int t = threadIdx.x; t < max_tiles; t += blockDim.x) tile_group[t] = -1;
     __syncthreads();
-    for (int p = threadIdx.x; p < pairs; p += blockDim.x) pair_pos[p] = atomicAdd(&cnt[idx[p]], 1);   // rank inside its expert
+    for (int p = threadIdx.x; p < pairs; p += blockDim.x)
+        pair_pos[p] = idx[p] >= 0 ? atomicAdd(&cnt[idx[p]], 1) : -1;   // rank inside its expert
     __syncthreads();
     if (threadIdx.x == 0) {
         int o = 0;
@@ -117,6 +123,7 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int32_t* __restric
     for (int e = threadIdx.x; e < experts; e += blockDim.x)
         for (int t = off[e] / tile; t < (off[e] + cnt[e] + tile - 1) / tile; ++t) tile_group[t] = e;
     for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+        if (idx[p] < 0) continue;
         const int pos = off[idx[p]] + pair_pos[p];
         pair_pos[p] = pos;
         src_row[pos] = p / top;
@@ -148,17 +155,17 @@ __global__ void gather_rows_bf16_kernel(const float* __restrict__ A, int64_t lda
     }
 }
 
-// x[r] += alpha * sum_k w[r, k] * y[pair_pos[r * top + k]] (pair_pos null: position = pair)
+// x[r] += alpha * sum_k w[r, k] * y[pair_pos[r * top + k]] (a negative position: h[r] in y's place)
 __global__ void moe_combine_kernel(float* __restrict__ x, const float* __restrict__ y, int64_t ldy, const int32_t* __restrict__ pair_pos,
-                                   const float* __restrict__ w, int top, int cols, float alpha) {
+                                   const float* __restrict__ w, int top, int cols, float alpha, const float* __restrict__ h, int64_t ldh) {
     const size_t r = blockIdx.y;
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= cols) return;
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
         const size_t p = r * top + k;
-        const size_t pos = pair_pos != nullptr ? (size_t)pair_pos[p] : p;
-        acc = fmaf(w[p], y[pos * ldy + c], acc);
+        const int pos = pair_pos[p];
+        acc = fmaf(w[p], pos >= 0 ? y[(size_t)pos * ldy + c] : h[r * ldh + c], acc);
     }
     x[r * cols + c] += alpha * acc;
 }
@@ -170,7 +177,8 @@ int moe_route_f32(const MoeRouteArgs& a, cudaStream_t st) {
     B2_CHECK_ARG(a.groups >= 1 && a.experts % a.groups == 0 && a.keep >= 1 && a.keep <= a.groups, "moe_route: %d experts in %d groups, %d kept", a.experts,
                  a.groups, a.keep);
     const int warps = 4;
-    const size_t smem = (size_t)warps * (2 * a.experts + a.groups) * sizeof(float);
+    B2_CHECK_ARG(a.identity >= 0 && a.identity < a.experts, "moe_route: %d identity experts of %d", a.identity, a.experts);
+    const size_t smem = (size_t)warps * (3 * a.experts + a.groups) * sizeof(float);
     B2_CHECK_ARG(smem <= 48 * 1024, "moe_route: %d experts exceed the router kernel's shared memory", a.experts);
     moe_route_kernel<<<(a.rows + warps - 1) / warps, warps * 32, smem, st>>>(a);
     B2_LAUNCH_CHECK();
@@ -194,10 +202,6 @@ int glu_rows_f32(const float* in, int64_t ld_in, float* out, int64_t ld_out, int
     return 0;
 }
 
-int swiglu_rows_f32(const float* in, int64_t ld_in, float* out, int64_t ld_out, int rows, int ff, cudaStream_t st, void* out16, int64_t ld_out16) {
-    return glu_rows_f32(in, ld_in, out, ld_out, rows, ff, GluAct{}, st, out16, ld_out16);
-}
-
 int gather_rows_bf16(const float* A, int64_t lda, const int32_t* src_row, void* out, int64_t ld_out, int rows, int K, cudaStream_t st) {
     B2_CHECK_ARG(A && src_row && out && rows > 0 && K > 0 && ld_out % 2 == 0, "gather_rows_bf16: bad argument");
     gather_rows_bf16_kernel<<<dim3((K / 2 + 256) / 256, rows), 256, 0, st>>>(A, lda, src_row, reinterpret_cast<__nv_bfloat16*>(out), ld_out, K);
@@ -206,9 +210,9 @@ int gather_rows_bf16(const float* A, int64_t lda, const int32_t* src_row, void* 
 }
 
 int moe_combine_f32(float* x, const float* y, int64_t ldy, const int32_t* pair_pos, const float* w, int rows, int top, int cols, float alpha,
-                    cudaStream_t st) {
-    B2_CHECK_ARG(x && y && w && rows > 0 && top > 0 && cols > 0, "moe_combine: bad argument");
-    moe_combine_kernel<<<dim3((cols + 255) / 256, rows), 256, 0, st>>>(x, y, ldy, pair_pos, w, top, cols, alpha);
+                    cudaStream_t st, const float* h, int64_t ldh) {
+    B2_CHECK_ARG(x && y && w && pair_pos && rows > 0 && top > 0 && cols > 0, "moe_combine: bad argument");
+    moe_combine_kernel<<<dim3((cols + 255) / 256, rows), 256, 0, st>>>(x, y, ldy, pair_pos, w, top, cols, alpha, h, ldh);
     B2_LAUNCH_CHECK();
     return 0;
 }

@@ -202,7 +202,7 @@ __global__ void rms_scalar_kernel(float* __restrict__ x, const int32_t* __restri
 
 // weighted RMS norm of a (gathered) row; accumulate: added onto out
 __global__ void rms_weight_kernel(const float* __restrict__ in, int64_t ld_in, const int32_t* __restrict__ row_index, const float* __restrict__ w,
-                                  float* __restrict__ out, int64_t ld_out, int accumulate, int cols, float eps) {
+                                  float* __restrict__ out, int64_t ld_out, int accumulate, int cols, float eps, __nv_bfloat16* __restrict__ out16) {
     __shared__ float red[33];
     const size_t r = blockIdx.x;
     const float* xr = in + (row_index != nullptr ? (size_t)row_index[r] : r) * ld_in;
@@ -213,7 +213,69 @@ __global__ void rms_weight_kernel(const float* __restrict__ in, int64_t ld_in, c
     for (int c = threadIdx.x; c < cols; c += blockDim.x) {
         const float v = xr[c] * mul * w[c];
         o[c] = accumulate ? o[c] + v : v;
+        if (out16 != nullptr) out16[r * cols + c] = __float2bfloat16_rn(v);
     }
+}
+
+// the same for rows of whole 16-byte pieces, at most V per thread: a row is read once, stays in registers, and its weights are loaded in
+// front of the reduction (in and out may be the same rows)
+template <int V>
+__global__ void __launch_bounds__(256) rms_weight_reg_kernel(const float* in, int64_t ld_in, const int32_t* __restrict__ row_index,
+                                                             const float* __restrict__ w, float* out, int64_t ld_out, int accumulate, int cols, float eps,
+                                                             __nv_bfloat16* __restrict__ out16) {
+    __shared__ float red[33];
+    const size_t r = blockIdx.x;
+    const float* xr = in + (row_index != nullptr ? (size_t)row_index[r] : r) * ld_in;
+    float4 x[V], g[V];
+    float q = 0.f;
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int c = (threadIdx.x + u * blockDim.x) * 4;
+        x[u] = g[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < cols) {
+            x[u] = *reinterpret_cast<const float4*>(xr + c);
+            g[u] = *reinterpret_cast<const float4*>(w + c);
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        q = fmaf(x[u].x, x[u].x, q); q = fmaf(x[u].y, x[u].y, q);
+        q = fmaf(x[u].z, x[u].z, q); q = fmaf(x[u].w, x[u].w, q);
+    }
+    const float mul = 1.f / sqrtf(block_sum(q, red) / (float)cols + eps);
+    float* o = out + r * ld_out;
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int c = (threadIdx.x + u * blockDim.x) * 4;
+        if (c >= cols) continue;
+        float4 v = make_float4(x[u].x * mul * g[u].x, x[u].y * mul * g[u].y, x[u].z * mul * g[u].z, x[u].w * mul * g[u].w);
+        if (out16 != nullptr) {
+            __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(out16 + r * cols + c);
+            h[0] = __floats2bfloat162_rn(v.x, v.y);
+            h[1] = __floats2bfloat162_rn(v.z, v.w);
+        }
+        if (accumulate) {
+            const float4 p = *reinterpret_cast<const float4*>(o + c);
+            v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
+        }
+        *reinterpret_cast<float4*>(o + c) = v;
+    }
+}
+
+// token row -> weighted RMS norm of the table's row (the residual stream of a model whose embedding is normed)
+template <typename TT>
+__global__ void embed_norm_kernel(const int32_t* __restrict__ tokens, const TT* __restrict__ table, float* __restrict__ x, int cols, int vocab,
+                                  int* err_flag, const float* __restrict__ w, float eps) {
+    __shared__ float red[33];
+    const size_t r = blockIdx.x;
+    const int t = tokens[r];
+    const bool ok = t >= 0 && t < vocab;
+    if (!ok && threadIdx.x == 0 && err_flag != nullptr) err_flag[0] = 1;  // slot 0 = B2_ERR_TOKEN_RANGE
+    const TT* e = table + (size_t)(ok ? t : 0) * cols;
+    float q = 0.f;
+    for (int c = threadIdx.x; c < cols; c += blockDim.x) q = fmaf((float)e[c], (float)e[c], q);
+    const float mul = ok ? 1.f / sqrtf(block_sum(q, red) / (float)cols + eps) : 0.f;
+    for (int c = threadIdx.x; c < cols; c += blockDim.x) x[r * cols + c] = (float)e[c] * mul * w[c];
 }
 
 // post-norm add of one sublayer, pre-norm of the next, and (decode steps) the input convolution with its carried inputs
@@ -535,8 +597,17 @@ int diff_combine_f32(const float* y, int64_t ldy, float* out, int64_t ldo, int r
 }
 
 int embed_rows_f32(const int32_t* tokens, const void* table, int table_dtype, float* x, int rows, int cols, int vocab, int* err_flag,
-                   cudaStream_t st, float scale) {
-    B2_CHECK_ARG(tokens && table && x && rows > 0, "embed_rows: bad argument");
+                   cudaStream_t st, float scale, const float* norm_w, float eps) {
+    B2_CHECK_ARG(tokens && table && x && rows > 0 && (norm_w == nullptr || scale == 1.f), "embed_rows: bad argument");
+    if (norm_w != nullptr) {
+        const int threads = cols >= 1024 ? 256 : 128;
+        if (table_dtype == DT_F32)
+            embed_norm_kernel<float><<<rows, threads, 0, st>>>(tokens, reinterpret_cast<const float*>(table), x, cols, vocab, err_flag, norm_w, eps);
+        else
+            embed_norm_kernel<__nv_bfloat16><<<rows, threads, 0, st>>>(tokens, reinterpret_cast<const __nv_bfloat16*>(table), x, cols, vocab, err_flag, norm_w, eps);
+        B2_LAUNCH_CHECK();
+        return 0;
+    }
     if (table_dtype == DT_F32)
         embed_rows_kernel<float><<<rows, 128, 0, st>>>(tokens, reinterpret_cast<const float*>(table), x, cols, vocab, err_flag, scale);
     else
@@ -561,9 +632,18 @@ int rms_scalar_f32(float* x, const int32_t* row_index, const float* g, const flo
 }
 
 int rms_weight_f32(const float* in, int64_t ld_in, const int32_t* row_index, const float* w, float* out, int64_t ld_out, int accumulate, int rows,
-                   int cols, float eps, cudaStream_t st) {
-    B2_CHECK_ARG(in && w && out && rows > 0 && cols > 0, "rms_weight: bad argument");
-    rms_weight_kernel<<<rows, cols >= 1024 ? 256 : 128, 0, st>>>(in, ld_in, row_index, w, out, ld_out, accumulate, cols, eps);
+                   int cols, float eps, cudaStream_t st, void* out16) {
+    B2_CHECK_ARG(in && w && out && rows > 0 && cols > 0 && (out16 == nullptr || !accumulate), "rms_weight: bad argument");
+    __nv_bfloat16* o16 = reinterpret_cast<__nv_bfloat16*>(out16);
+    const uintptr_t align = reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(out16);
+    if (cols % 4 == 0 && ld_in % 4 == 0 && ld_out % 4 == 0 && (align & 15) == 0 && cols <= 8192) {
+        if (cols <= 512) rms_weight_reg_kernel<1><<<rows, 128, 0, st>>>(in, ld_in, row_index, w, out, ld_out, accumulate, cols, eps, o16);
+        else if (cols <= 2048) rms_weight_reg_kernel<2><<<rows, 256, 0, st>>>(in, ld_in, row_index, w, out, ld_out, accumulate, cols, eps, o16);
+        else if (cols <= 4096) rms_weight_reg_kernel<4><<<rows, 256, 0, st>>>(in, ld_in, row_index, w, out, ld_out, accumulate, cols, eps, o16);
+        else rms_weight_reg_kernel<8><<<rows, 256, 0, st>>>(in, ld_in, row_index, w, out, ld_out, accumulate, cols, eps, o16);
+    } else {
+        rms_weight_kernel<<<rows, cols >= 1024 ? 256 : 128, 0, st>>>(in, ld_in, row_index, w, out, ld_out, accumulate, cols, eps, o16);
+    }
     B2_LAUNCH_CHECK();
     return 0;
 }

@@ -2,7 +2,7 @@
 // (m, m + pairs)) turn by position * f_m.
 // cos and sin come from a table [position][pair] that the cache builds on the host in double precision (the plain
 // frequencies base^(-2m/dims), optionally blended towards f_m / factor over a ramp of pairs with cos / sin scaled, the long-context
-// form known as YaRN, or scaled by bands of wavelength), so an angle never carries the rounding of a 32-bit product of a large position. One kernel serves
+// form known as YaRN, scaled by bands of wavelength, or all divided by one factor), so an angle never carries the rounding of a 32-bit product of a large position. One kernel serves
 // queries (in place), keys and values on their way into the cache slabs, a rotated part copied to another layout, and the
 // turn back of an attention output by its query's position with the sigmoid output gate applied in the same pass. When a head is
 // normed before it turns (weighted RMS norm over the head, one weight vector for all heads), one warp takes a (row, head): it sums
@@ -233,6 +233,10 @@ void rotary_frequencies(const RotaryDesc& d, std::vector<double>& freq, double& 
     for (int i = 0; i < pairs; ++i) freq[i] = pow((double)d.base, -2.0 * i / d.dims);
     if (!(d.factor > 0.f)) return;
     const double two_pi = 6.283185307179586476925286766559;
+    if (d.scaling == ROT_LINEAR) {
+        for (double& f : freq) f /= d.factor;
+        return;
+    }
     if (d.scaling == ROT_BANDS) {
         for (int i = 0; i < pairs; ++i) {
             const double turns = d.original * freq[i] / two_pi;   // original / wavelength

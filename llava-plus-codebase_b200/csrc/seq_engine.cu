@@ -32,6 +32,8 @@ struct SeqWeights {   // tensors of one layer that owns its weights
     float lambda = 0.f;                                 // differential attention and the layer's lambda (made from them when the model is finalized)
     DevBuf gla_w, a2_w, a2_b, gnorm;                    // gated linear attention: [q | k | v | g | a1] fused, W_a2 and its bias, the heads' norm weight
     DevBuf norm1_a, norm2_a;                            // dynamic tanh: the norms' slopes (one number each; the bias lies in norm1_b / norm2_b)
+    DevBuf qkv_b, qkv_b16;                              // grouped attention: biases of q, k, v in front of zeros for the gate (fp32; bf16: GEMM epilogue)
+    DevBuf router_c;                                    // experts: correction of the choice scores
     DevBuf mem_w, mnorm_w, gate1_b, gate2_b;            // matrix memories: [q | k | v | two gates | g] fused, norm weight, biases of the gates (mLSTM:
                                                         // input, forget; the delta rule's decay bias and logarithm lie in dt_bias / a_log)
     std::map<std::string, int> got;
@@ -60,7 +62,7 @@ struct SeqModel {
     std::vector<SeqLayerInfo> layers;
     std::vector<SeqRun> runs;          // what one forward pass executes, in order (a looped layer appears once per pass)
     std::vector<SeqWeights> w;
-    DevBuf embed, head, final_w, final_b, final_a;
+    DevBuf embed, head, final_w, final_b, final_a, embed_nw;
     DevBuf bigram, loop_step;          // [buckets + 1, width] in the weight dtype; [times, width] fp32
     DevBuf x0;                         // the embedding output, kept for the passes of a looped block
     DevBuf loop_in, cat;               // looped block with an input mix: W_in [width, 2 width], rows [x | x0] in fp32
@@ -204,6 +206,8 @@ struct Lin {  // one Linear call on the model's compute dtype
         return linear_f32(a, st);
     }
 };
+
+bool is_glu(int ff_kind) { return ff_kind == B2_FF_CLAMP_GLU || ff_kind == B2_FF_GELU_GLU; }   // one dense pair [gate | up] around a gated unit
 
 int router_rows(int experts) { return std::max(32, (experts + 7) / 8 * 8); }   // rows of the (zero-padded) router matrix
 
@@ -350,7 +354,7 @@ static int latent_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeight
     return lin(y, L.pv, W.o_w, width, L.pv, target, width, R, LIN_NONE, alpha, accumulate);
 }
 
-// Attention with grouped key/value heads, a short convolution on q / k / v, an optional weighted norm of the q / k heads, rotary q / k in
+// Attention with grouped key/value heads, biases on q / k / v, a short convolution on q / k / v, an optional weighted norm of the q / k heads, rotary q / k in
 // either pair layout, optionally rotated values, a masked softmax with an optional fixed sink, and a sigmoid output gate per channel or
 // per head. With two maps (differential attention) the projection rows were ordered [map][head][dim] when the tensors were set, so the
 // maps are simply twice the query and key heads over the same value heads, and a head's two outputs are joined after the softmax.
@@ -367,7 +371,7 @@ static int gqa_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeights& 
     const int32_t* row_slot = s.row_slot.as<int32_t>();
     const int32_t* row_pos = s.row_pos.as<int32_t>();
     float* proj = s.proj.as<float>();  // [R, nq | nk | nv | gate]
-    B2_TRY(lin(in.h, width, W.lproj_w, L.lproj, width, proj, L.lproj_ld, R, LIN_NONE, 1.f, 0, nullptr, 0, nullptr, in.h16, in.norm));
+    B2_TRY(lin(in.h, width, W.lproj_w, L.lproj, width, proj, L.lproj_ld, R, LIN_NONE, 1.f, 0, W.qkv_b.as<float>(), 0, W.qkv_b16.p, in.h16, in.norm));
     float* qkv = proj;
     int64_t ldc = L.lproj_ld;
     if (d.ga_conv >= 1) {
@@ -406,14 +410,20 @@ static int gqa_mixer(b2_model* m, b2_kv* kv, const SeqLayerInfo& L, SeqWeights& 
     // one sigmoid per head rides in the attention's last write (unless the head's output is still to be joined or turned back)
     const bool gate_in_attn = d.ga_gate == B2_GATE_HEAD && maps == 1 && !d.ga_rot_values;
     if (gate_in_attn) { aa.head_gate = gates; aa.ldg = L.lproj_ld; }
+    // so does a sigmoid per channel, and the output leaves as the bf16 operand of W_o when that product runs on the tensor cores
+    const bool chan_in_attn = d.ga_gate == B2_GATE_CHANNEL && maps == 1 && !d.ga_rot_values;
+    if (chan_in_attn) { aa.chan_gate = gates; aa.ldg = L.lproj_ld; }
+    const bool out16 = maps == 1 && !d.ga_rot_values && lin.tensor_cores(width, L.ng, target, width, R);
+    if (out16) aa.out16 = s.a16.p;
     B2_TRY(attn_bias_f32(aa, st));
+    if (out16) return lin(nullptr, 0, W.o_w, width, L.ng, target, width, R, LIN_NONE, alpha, accumulate, nullptr, 0, nullptr, s.a16.p);
     const float* yo = s.y.as<float>();
     float* gated = s.gated.as<float>();
     if (maps > 1) {   // a head's two maps: unit_rms(a1 - lambda a2) * (1 - diff)
         B2_TRY(diff_combine_f32(yo, (int64_t)maps * L.ng, gated, L.ng, R, H, dv, W.lambda, 1.f - d.ga_diff, s.d.norm_eps, st));
         yo = gated;
     }
-    if (d.ga_rot_values || d.ga_gate == B2_GATE_CHANNEL) {
+    if (d.ga_rot_values || (d.ga_gate == B2_GATE_CHANNEL && !chan_in_attn)) {
         // every head's output is turned back by the query's position, and the per-channel sigmoid gate is applied in the same pass
         RotateArgs rb;
         rb.in = yo; rb.ld_in = L.ng; rb.hs_in = dv; rb.out = gated; rb.ld_out = L.ng; rb.hs_out = dv;
@@ -573,9 +583,16 @@ static int parallel_inputs(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, fl
     const int width = s.d.width;
     const float eps = s.d.norm_eps;
     float* xn = s.xn.as<float>();
+    // the sublayers whose first product takes a SubIn in all its forms (the others read fp32 rows)
+    const bool mixer_ok = L.d.type == B2_MIXER_GQA_ATTN || L.d.type == B2_MIXER_MLSTM || L.d.type == B2_MIXER_DELTA;
+    const int Np = (N1 + 7) / 8 * 8;
     if (s.d.norm_kind != B2_NORM_DYT) {
-        B2_TRY(rms_weight_f32(x, width, nullptr, W.norm1.as<float>(), xn, width, 0, R, width, eps, st));
-        in1 = in2 = SubIn(xn);
+        // a rounded copy beside the fp32 rows where the first product reads bf16 (the other products of both sublayers then read it too)
+        void* h16 = mixer_ok && lin.tensor_cores(N1, width, s.proj.as<float>(), Np, R, W.qkv_b.as<float>(), 0, W.qkv_b16.p) ? s.h1_16.p : nullptr;
+        B2_TRY(rms_weight_f32(x, width, nullptr, W.norm1.as<float>(), xn, width, 0, R, width, eps, st, h16));
+        in1 = SubIn(xn);
+        in1.h16 = h16;
+        in2 = in1;
         if (two) {
             B2_TRY(rms_weight_f32(x, width, nullptr, W.norm2.as<float>(), s.h2.as<float>(), width, 0, R, width, eps, st));
             in2 = SubIn(s.h2.as<float>());
@@ -584,8 +601,6 @@ static int parallel_inputs(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, fl
     }
     n1 = dyt_of(W.norm1_a, W.norm1, W.norm1_b);
     if (two) n2 = dyt_of(W.norm2_a, W.norm2, W.norm2_b);
-    // the sublayers whose first product takes a SubIn in all its forms (the others read fp32 rows)
-    const bool mixer_ok = L.d.type == B2_MIXER_GQA_ATTN || L.d.type == B2_MIXER_MLSTM || L.d.type == B2_MIXER_DELTA;
     const bool ff_ok = L.d.ff == 0 || L.d.ff_kind == B2_FF_GELU;
     if (lin.fuses_norm(width, R) && mixer_ok && ff_ok) {
         in1.h = in2.h = x;
@@ -593,7 +608,6 @@ static int parallel_inputs(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, fl
         if (two) in2.norm = &n2;
         return 0;
     }
-    const int Np = (N1 + 7) / 8 * 8;
     const bool tc1 = mixer_ok && lin.tensor_cores(N1, width, s.proj.as<float>(), Np, R) && (two || L.d.ff == 0);
     const bool tc2 = two && L.d.ff_kind == B2_FF_GELU && gelu_on_tensor_cores(s, lin, L.d.ff, target, R);
     DytOut o[2];
@@ -633,9 +647,10 @@ static int sandwich_input(SeqModel& s, const float* post, const DevBuf& norm, co
     return 0;
 }
 
-// The feed-forward of a pre-norm or sandwich block in its three kinds.
-static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, const float* h, float* target, float alpha, int accumulate, int R,
+// The feed-forward of a pre-norm, sandwich or parallel block in its kinds. in.h holds the fp32 rows always, in.h16 their rounded copy sometimes.
+static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, const SubIn& in, float* target, float alpha, int accumulate, int R,
                             cudaStream_t st) {
+    const float* h = in.h;
     SeqModel& s = *m->seq;
     const b2_seq_layer_desc& d = L.d;
     const Lin lin{m, st};
@@ -647,20 +662,22 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
         B2_TRY(polynorm_f32(s.ff.as<float>(), ffl, W.up_b.as<float>(), W.act_coef.as<float>(), s.ffa.as<float>(), d.ff, R, d.ff, eps, st));
         return lin(s.ffa.as<float>(), d.ff, W.down_w, width, d.ff, target, width, R, LIN_NONE, alpha, accumulate, W.down_b.as<float>(), 0, W.down_b16.p);
     }
-    if (d.ff_kind == B2_FF_CLAMP_GLU) {
-        // [gate | up] in one matrix; the bounded gated unit a(g) (u + 1); a decode step of one row takes product and unit in one launch (more rows would
+    const GluAct clamp_glu{d.ff_act_slope, d.ff_limit, 1.f};   // the bounded gated unit a(g) (u + 1)
+    if (is_glu(d.ff_kind)) {
+        // [gate | up] in one matrix, then the gated unit; a decode step of one row takes product and unit in one launch (more rows would
         // stream the matrix once per row there)
         const int ff = d.ff, ffl = (2 * ff + 7) / 8 * 8;
-        const GluAct act{d.ff_act_slope, d.ff_limit, 1.f};
+        GluAct act = clamp_glu;
+        if (d.ff_kind == B2_FF_GELU_GLU) { act = GluAct{}; act.kind = GLU_GELU_TANH; }
         if (R == 1) {
             GroupedLinearArgs gs;
             gs.A = h; gs.lda = width; gs.a_div = 1; gs.W = W.up_w.p; gs.ldw = width; gs.w_group_stride = 0; gs.w_dtype = s.w_dtype;
             gs.tile_group = s.zero_idx.as<int32_t>(); gs.tile_rows = 1; gs.out = s.ffa.as<float>(); gs.ld_out = ff;
             gs.M = R; gs.N = ff; gs.K = width; gs.round_a = s.d.compute == B2_COMPUTE_BF16; gs.swiglu = 1;
-            gs.glu_slope = act.slope; gs.glu_limit = act.limit; gs.glu_up_shift = act.up_shift;
+            gs.glu = act;
             B2_TRY(linear_grouped_f32(gs, st));
         } else {
-            B2_TRY(lin(h, width, W.up_w, 2 * ff, width, s.ff.as<float>(), ffl, R));
+            B2_TRY(lin(h, width, W.up_w, 2 * ff, width, s.ff.as<float>(), ffl, R, LIN_NONE, 1.f, 0, nullptr, 0, nullptr, in.h16));
             if (lin.tensor_cores(width, ff, target, width, R)) {   // the unit writes the bf16 rows that the second product reads
                 B2_TRY(glu_rows_f32(s.ff.as<float>(), ffl, nullptr, 0, R, ff, act, st, s.a16.p, ff));
                 return lin(nullptr, 0, W.down_w, width, ff, target, width, R, LIN_NONE, alpha, accumulate, nullptr, 0, nullptr, s.a16.p);
@@ -670,7 +687,7 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
         return lin(s.ffa.as<float>(), ff, W.down_w, width, ff, target, width, R, LIN_NONE, alpha, accumulate);
     }
     if (d.ff_kind == B2_FF_GELU) {
-        B2_TRY(gelu_up(m, L, W, SubIn(h), target, R, st));
+        B2_TRY(gelu_up(m, L, W, in, target, R, st));
         return gelu_down(m, L, W, target, alpha, accumulate, R, st);
     }
     if (d.ff_kind != B2_FF_MOE) {
@@ -678,12 +695,15 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
         return lin(s.ff.as<float>(), (d.ff + 7) / 8 * 8, W.down_w, width, d.ff, target, width, R, LIN_NONE, alpha, accumulate);
     }
     const int E = d.moe_experts, top = d.moe_top, ff = d.ff;
-    const bool gated = d.moe_act == B2_MOE_ACT_SWIGLU;
+    const bool gated = d.moe_act != B2_MOE_ACT_RELU_SQ;
+    const GluAct act = d.moe_act == B2_MOE_ACT_CLAMP_GLU ? clamp_glu : GluAct{};   // the experts' gated unit
     const int un = gated ? 2 * ff : ff;   // rows of an expert's first matrix: [gate | up], or up alone
     const int round_a = s.d.compute == B2_COMPUTE_BF16;
-    B2_TRY(lin(h, width, W.router_w, router_rows(E), width, s.rlogit.as<float>(), router_rows(E), R));
+    const int choices = E + d.moe_identity;   // rows of the router: the experts, then the identity experts
+    B2_TRY(lin(h, width, W.router_w, router_rows(choices), width, s.rlogit.as<float>(), router_rows(choices), R, LIN_NONE, 1.f, 0, nullptr, 0, nullptr, in.h16));
     MoeRouteArgs ra;
-    ra.logits = s.rlogit.as<float>(); ra.ld = router_rows(E); ra.rows = R; ra.experts = E; ra.top = top;
+    ra.logits = s.rlogit.as<float>(); ra.ld = router_rows(choices); ra.rows = R; ra.experts = choices; ra.top = top;
+    ra.identity = d.moe_identity; ra.correction = W.router_c.as<float>();
     ra.groups = d.moe_groups; ra.keep = d.moe_keep; ra.scale = d.moe_scale;
     ra.score_fn = d.moe_score; ra.group_score = d.moe_group_score; ra.raw_weights = d.moe_raw_weights;
     ra.idx = s.moe_idx.as<int32_t>(); ra.w = s.moe_w.as<float>();
@@ -700,11 +720,11 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
                 GroupedLinearArgs gs;
                 gs.A = h; gs.lda = width; gs.a_div = 1; gs.W = W.sgu_w.p; gs.ldw = width; gs.w_group_stride = 0; gs.w_dtype = s.w_dtype;
                 gs.tile_group = s.zero_idx.as<int32_t>(); gs.tile_rows = 1; gs.out = s.ffa.as<float>(); gs.ld_out = sf;
-                gs.M = R; gs.N = sf; gs.K = width; gs.round_a = round_a; gs.swiglu = 1;
+                gs.M = R; gs.N = sf; gs.K = width; gs.round_a = round_a; gs.swiglu = 1; gs.glu = act;
                 B2_TRY(linear_grouped_f32(gs, st));
             } else {
                 B2_TRY(lin(h, width, W.sgu_w, 2 * sf, width, s.ff.as<float>(), sfl, R));
-                B2_TRY(swiglu_rows_f32(s.ff.as<float>(), sfl, s.ffa.as<float>(), sf, R, sf, st));
+                B2_TRY(glu_rows_f32(s.ff.as<float>(), sfl, s.ffa.as<float>(), sf, R, sf, act, st));
             }
             B2_TRY(lin(s.ffa.as<float>(), sf, W.sd_w, width, sf, target, width, R, LIN_NONE, alpha, accumulate));
         }
@@ -722,7 +742,14 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
     const bool tc = ga.round_a && R >= 64 && tc_enabled() && width % 8 == 0 && ff % 8 == 0 && width >= 32 && ff >= 32;
     if (R <= 8) {   // decode step: gate, up and the gated activation of a pair in one launch
         ga.tile_rows = 1; ga.tile_group = s.moe_idx.as<int32_t>(); ga.a_div = top; ga.M = P;
-        if (gated) { ga.swiglu = 1; ga.N = ff; ga.out = s.moe_a.as<float>(); ga.ld_out = ff; }
+        if (gated) { ga.swiglu = 1; ga.glu = act; ga.N = ff; ga.out = s.moe_a.as<float>(); ga.ld_out = ff; }
+        B2_TRY(linear_grouped_f32(ga, st));
+        // second products and the weighted sum over a token's choices, onto the target
+        ExpertSumArgs es;
+        es.a = s.moe_a.as<float>(); es.lda = ff; es.W = W.ed_w.p; es.w_group_stride = (int64_t)width * ff; es.w_dtype = s.w_dtype;
+        es.idx = s.moe_idx.as<int32_t>(); es.w = s.moe_w.as<float>(); es.h = h; es.ldh = width; es.x = target; es.ldx = width;
+        es.rows = R; es.top = top; es.N = width; es.K = ff; es.round_a = round_a; es.alpha = alpha;
+        return expert_sum_f32(es, st);
     } else {
         const int tile = tc ? 128 : GROUPED_TILE_ROWS;
         const int tiles = (R * top + E * (tile - 1) + tile - 1) / tile;
@@ -743,7 +770,7 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
         g1.M = P; g1.N = un; g1.K = width; g1.tile_group = s.moe_tile.as<int32_t>(); g1.groups = E;
         if (!gated) g1.post = LIN_RELU_SQ;
         B2_TRY(gemm_bf16(g1, st));
-        if (gated) B2_TRY(swiglu_rows_f32(s.moe_h.as<float>(), 2 * ff, nullptr, 0, P, ff, st, h16, ff));
+        if (gated) B2_TRY(glu_rows_f32(s.moe_h.as<float>(), 2 * ff, nullptr, 0, P, ff, act, st, h16, ff));
         else B2_TRY(cast_rows_bf16(s.moe_h.as<float>(), ff, h16, ff, P, ff, st));
         GemmArgs g2;
         g2.A = h16; g2.lda = ff; g2.W = W.ed_w.p; g2.ldw = ff; g2.out = s.moe_y.p; g2.ld_out = width; g2.out_fp32 = 1;
@@ -751,15 +778,15 @@ static int seq_feed_forward(b2_model* m, const SeqLayerInfo& L, SeqWeights& W, c
         B2_TRY(gemm_bf16(g2, st));
     } else {
         B2_TRY(linear_grouped_f32(ga, st));
-        if (gated && !ga.swiglu) B2_TRY(swiglu_rows_f32(s.moe_h.as<float>(), 2 * ff, s.moe_a.as<float>(), ff, P, ff, st));
+        if (gated) B2_TRY(glu_rows_f32(s.moe_h.as<float>(), 2 * ff, s.moe_a.as<float>(), ff, P, ff, act, st));
         GroupedLinearArgs gd = ga;
-        gd.swiglu = 0; gd.act = LIN_NONE;
+        gd.act = LIN_NONE;
         gd.A = s.moe_a.as<float>(); gd.lda = ff; gd.a_rows = nullptr; gd.a_div = 1;
         gd.W = W.ed_w.p; gd.ldw = ff; gd.w_group_stride = (int64_t)width * ff;
         gd.out = s.moe_y.as<float>(); gd.ld_out = width; gd.N = width; gd.K = ff;
         B2_TRY(linear_grouped_f32(gd, st));
     }
-    return moe_combine_f32(target, s.moe_y.as<float>(), width, pos, s.moe_w.as<float>(), R, top, width, alpha, st);
+    return moe_combine_f32(target, s.moe_y.as<float>(), width, pos, s.moe_w.as<float>(), R, top, width, alpha, st, h, width);
 }
 
 // ------------------------------------------------------------------------------------------------------------------
@@ -822,7 +849,7 @@ static int seq_forward(b2_model* m, b2_kv* kv, int R, int nseg, int slot, int ct
                     B2_TRY(hgrn2_mixer(m, L, W, S, in1.h, x, rm, 1, R, nseg, st));
                 }
                 if (early) B2_TRY(gelu_down(m, L, W, x, rm, 1, R, st));
-                else if (d.ff > 0) B2_TRY(seq_feed_forward(m, L, W, in2.h, x, rm, 1, R, st));
+                else if (d.ff > 0) B2_TRY(seq_feed_forward(m, L, W, in2, x, rm, 1, R, st));
                 if (resid_out != nullptr)
                     B2_CUDA_CHECK(cudaMemcpyAsync(resid_out + ri * (size_t)R * width, x, (size_t)R * width * F4, cudaMemcpyDeviceToDevice, st));
                 continue;
@@ -949,7 +976,8 @@ static int seq_embed(b2_model* m, b2_kv* kv, const int32_t* tokens, int R, int n
         return embed_bigram_rows_f32(tokens, s.segs.as<SeqSeg>(), nseg, nseg == 1 ? R : 1, s.embed.p, s.bigram.p, s.w_dtype, kv->seq->last_tok.as<int32_t>(),
                                      s.x.as<float>(), s.x0.as<float>(), s.d.width, s.d.vocab, s.d.bigram_buckets, s.d.bigram_mul_prev, s.d.bigram_mul_cur,
                                      m->err_dev, st);
-    return embed_rows_f32(tokens, s.embed.p, s.w_dtype, s.x.as<float>(), R, s.d.width, s.d.vocab, m->err_dev, st, s.d.embed_scale != 0.f ? s.d.embed_scale : 1.f);
+    return embed_rows_f32(tokens, s.embed.p, s.w_dtype, s.x.as<float>(), R, s.d.width, s.d.vocab, m->err_dev, st, s.d.embed_scale != 0.f ? s.d.embed_scale : 1.f,
+                          s.embed_nw.as<float>(), s.d.norm_eps);
 }
 
 // rows `index` (null: all) of x -> final norm -> head -> soft-cap: fp32 logits [n, vocab]
@@ -1027,6 +1055,7 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
         B2_TRY(want_shape(key, shape, ndim, s.d.loop_times, width)); s.got[k] = 1;
         return put_tensor(s.loop_step, DT_F32, (size_t)s.d.loop_times * width, 0, ptr, dt, (int64_t)s.d.loop_times * width);
     }
+    if (k == "embed.norm" && s.d.embed_norm) { B2_TRY(want_shape(key, shape, ndim, width)); s.got[k] = 1; return put_tensor(s.embed_nw, DT_F32, width, 0, ptr, dt, width); }
     if (k == "final.norm") { B2_TRY(want_shape(key, shape, ndim, width)); s.got[k] = 1; return put_tensor(s.final_w, DT_F32, width, 0, ptr, dt, width); }
     if (k == "final.norm.b") { B2_TRY(want_shape(key, shape, ndim, width)); s.got[k] = 1; return put_tensor(s.final_b, DT_F32, width, 0, ptr, dt, width); }
     int li = -1, used = 0;
@@ -1146,6 +1175,18 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
                 if (is_taps) return taps_of(W.conv_w, sizes[j], L.conv_ch, row0, d.ga_conv);
                 row0 += sizes[j];
             }
+            if (d.ga_qkv_bias) {
+                row0 = 0;
+                for (int j = 0; j < 3; ++j) {
+                    if (r == std::string(parts[j]) + ".b" && sizes[j] > 0) {
+                        B2_TRY(want_shape(key, shape, ndim, sizes[j]));
+                        W.got[r] = 1;
+                        B2_TRY(put_tensor(W.qkv_b, DT_F32, (size_t)(L.lproj + 7) / 8 * 8, row0, ptr, dt, sizes[j]));
+                        return put_tensor(W.qkv_b16, DT_BF16, (size_t)(L.lproj + 7) / 8 * 8, row0, ptr, dt, sizes[j]);
+                    }
+                    row0 += sizes[j];
+                }
+            }
             if (r == "mix.o") return mat(W.o_w, width, L.ng);
             if (d.ga_qk_norm) {
                 const bool all = d.ga_qk_norm == B2_QK_NORM_ALL;
@@ -1213,14 +1254,15 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
                 return put_tensor(W.down_b16, DT_BF16, (size_t)(width + 7) / 8 * 8, 0, ptr, dt, width);
             }
         } else if (d.ff > 0 && d.ff_kind == B2_FF_MOE) {
-            const int E = d.moe_experts, ff = d.ff, sf = d.moe_shared_ff;
-            const bool gated = d.moe_act == B2_MOE_ACT_SWIGLU;
+            const int E = d.moe_experts, choices = E + d.moe_identity, ff = d.ff, sf = d.moe_shared_ff;
+            const bool gated = d.moe_act != B2_MOE_ACT_RELU_SQ;
             const int un = gated ? 2 : 1;   // matrices in front of an expert's activation
             if (r == "mlp.router") {   // at least 32 rows (zeros behind the experts): the tensor-core product of a prompt portion takes it
-                B2_TRY(want_shape(key, shape, ndim, E, width));
+                B2_TRY(want_shape(key, shape, ndim, choices, width));
                 W.got[r] = 1;
-                return put_tensor(W.router_w, WD, (size_t)router_rows(E) * width, 0, ptr, dt, (int64_t)E * width);
+                return put_tensor(W.router_w, WD, (size_t)router_rows(choices) * width, 0, ptr, dt, (int64_t)choices * width);
             }
+            if (r == "mlp.correction" && d.moe_correction) return vec(W.router_c, choices);
             if (sf > 0) {
                 if (r == "mlp.shared.gate" && gated) return part(W.sgu_w, 2 * sf, 0, sf, width);
                 if (r == "mlp.shared.up") return part(W.sgu_w, un * sf, gated ? sf : 0, sf, width);
@@ -1242,7 +1284,7 @@ int seq_set_weight(b2_model* m, const char* key, const void* ptr, const int64_t*
                     return put_tensor(W.ed_w, WD, ((size_t)E * width + 8) * ff, (size_t)e * width * ff, ptr, dt, (int64_t)width * ff);
                 }
             }
-        } else if (d.ff > 0 && d.ff_kind == B2_FF_CLAMP_GLU) {
+        } else if (d.ff > 0 && is_glu(d.ff_kind)) {
             if (r == "mlp.gate") return part(W.up_w, 2 * d.ff, 0, d.ff, width);
             if (r == "mlp.up") return part(W.up_w, 2 * d.ff, d.ff, d.ff, width);
             if (r == "mlp.down") return mat(W.down_w, width, d.ff);
@@ -1332,6 +1374,7 @@ static std::vector<std::string> required_of(const SeqLayerInfo& L, const b2_seq_
             if (L.gw > 0) v.push_back("mix.g");
             if (d.ga_conv >= 1) for (const char* n : {"mix.q.conv", "mix.k.conv", "mix.v.conv"}) v.push_back(n);
             if (d.ga_qk_norm) for (const char* n : {"mix.q.norm", "mix.k.norm"}) v.push_back(n);
+            if (d.ga_qkv_bias) for (const char* n : {"mix.q.b", "mix.k.b", "mix.v.b"}) if (n[4] != 'v' || !d.ga_key_values) v.push_back(n);
             if (L.maps > 1) for (const char* n : {"mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"}) v.push_back(n);
         } else if (d.type == B2_MIXER_GLA) {
             for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.g", "mix.a1", "mix.a2", "mix.a2.b", "mix.norm"}) v.push_back(n);
@@ -1347,14 +1390,15 @@ static std::vector<std::string> required_of(const SeqLayerInfo& L, const b2_seq_
             if (L.d.ff_kind == B2_FF_POLYNORM) for (const char* n : {"mlp.up", "mlp.up.b", "mlp.down", "mlp.down.b", "mlp.act"}) v.push_back(n);
             else if (L.d.ff_kind == B2_FF_MOE) {
                 v.push_back("mlp.router");
-                const bool gated = L.d.moe_act == B2_MOE_ACT_SWIGLU;
+                if (L.d.moe_correction) v.push_back("mlp.correction");
+                const bool gated = L.d.moe_act != B2_MOE_ACT_RELU_SQ;
                 for (int e = 0; e < L.d.moe_experts; ++e)
                     for (const char* n : {"gate", "up", "down"})
                         if (gated || n[0] != 'g') v.push_back("mlp.e" + std::to_string(e) + "." + n);
                 if (L.d.moe_shared_ff > 0)
                     for (const char* n : {"mlp.shared.gate", "mlp.shared.up", "mlp.shared.down"})
                         if (gated || n[11] != 'g') v.push_back(n);
-            } else if (L.d.ff_kind == B2_FF_CLAMP_GLU) for (const char* n : {"mlp.gate", "mlp.up", "mlp.down"}) v.push_back(n);
+            } else if (is_glu(L.d.ff_kind)) for (const char* n : {"mlp.gate", "mlp.up", "mlp.down"}) v.push_back(n);
             else for (const char* n : {"mlp.up", "mlp.down"}) v.push_back(n);
         }
         return v;
@@ -1384,6 +1428,7 @@ int seq_finalize(b2_model* m) {
     if (dyt) top.push_back("final.norm.alpha");
     if (s.d.loop_mix) top.push_back("loop.in");
     if (s.d.bigram_buckets > 0) top.push_back("bigram");
+    if (s.d.embed_norm) top.push_back("embed.norm");
     if (s.d.loop_times >= 1 && !s.d.loop_plain && !s.d.loop_mix) top.push_back("loop.step");
     for (const std::string& n : top)
         if (!s.got.count(n) && missing.size() < 600) { missing += n; missing += ' '; }
@@ -1433,10 +1478,10 @@ int seq_finalize(b2_model* m) {
         }
         fw = std::max(fw, (L.d.ff + 7) / 8 * 8);
         if (L.d.ff > 0 && L.d.ff_kind == B2_FF_GELU) gelu = true;
-        if (L.d.ff > 0 && L.d.ff_kind == B2_FF_CLAMP_GLU) { fw = std::max(fw, (2 * L.d.ff + 7) / 8 * 8); glu = true; }
+        if (L.d.ff > 0 && is_glu(L.d.ff_kind)) { fw = std::max(fw, (2 * L.d.ff + 7) / 8 * 8); glu = true; }
         if (L.d.ff > 0 && L.d.ff_kind == B2_FF_MOE) {
             fw = std::max(fw, (2 * L.d.moe_shared_ff + 7) / 8 * 8);
-            moe_top = std::max(moe_top, L.d.moe_top); moe_e = std::max(moe_e, L.d.moe_experts); moe_ff = std::max(moe_ff, L.d.ff);
+            moe_top = std::max(moe_top, L.d.moe_top); moe_e = std::max(moe_e, L.d.moe_experts + L.d.moe_identity); moe_ff = std::max(moe_ff, L.d.ff);
         }
     }
 
@@ -1461,10 +1506,8 @@ int seq_finalize(b2_model* m) {
     if (s.d.block == B2_BLOCK_PARALLEL2) B2_TRY(s.h2.alloc(R * width * F4));
     if (den_w > 0) B2_TRY(s.den.alloc(R * den_w * F4));
     if (s.d.compute == B2_COMPUTE_BF16) {
-        if (dyt) {
-            B2_TRY(s.h1_16.alloc(R * width * 2));
-            B2_TRY(s.h2_16.alloc(R * width * 2));
-        }
+        if (dyt || s.d.block == B2_BLOCK_PARALLEL_RMS || s.d.block == B2_BLOCK_PARALLEL2) B2_TRY(s.h1_16.alloc(R * width * 2));
+        if (dyt) B2_TRY(s.h2_16.alloc(R * width * 2));
         if (gelu) B2_TRY(s.f16.alloc(R * fw * 2));
     }
     if (glu && moe_e == 0) {   // the one-row grouped product of a decode step reads its group (always 0) from here
@@ -1520,13 +1563,14 @@ void seq_model_free(b2_model* m) {
                         &W.lproj_w, &W.rel, &W.lo_w, &W.mu, &W.r_w, &W.k_w, &W.v_w, &W.g_w, &W.w1, &W.w2, &W.w0, &W.bonus, &W.rnorm, &W.ro_w,
                         &W.up_w, &W.down_w, &W.qdg_w, &W.dkv_norm, &W.uk_w, &W.ukT, &W.uv_w, &W.sink, &W.qfv_w, &W.f_b, &W.lower, &W.hnorm, &W.up_b, &W.down_b,
                         &W.down_b16, &W.act_coef, &W.router_w, &W.egu_w, &W.ed_w, &W.sgu_w, &W.sd_w, &W.canon1, &W.canon2, &W.dq_norm, &W.uq_w, &W.ukx_w,
-                        &W.qn_w, &W.kn_w, &W.lam4, &W.gla_w, &W.a2_w, &W.a2_b, &W.gnorm, &W.norm1_a, &W.norm2_a, &W.mem_w, &W.mnorm_w, &W.gate1_b, &W.gate2_b};
+                        &W.qn_w, &W.kn_w, &W.lam4, &W.gla_w, &W.a2_w, &W.a2_b, &W.gnorm, &W.norm1_a, &W.norm2_a, &W.mem_w, &W.mnorm_w, &W.gate1_b, &W.gate2_b,
+                        &W.qkv_b, &W.qkv_b16, &W.router_c};
         for (DevBuf* b : bs) b->free();
     }
     DevBuf* bs[] = {&s.embed, &s.head, &s.final_w, &s.final_b, &s.x, &s.proj, &s.act, &s.y, &s.gated, &s.mixout, &s.mixes, &s.rp, &s.wl1, &s.wlog,
                     &s.ff, &s.xn, &s.tok, &s.want, &s.segs, &s.row_slot, &s.row_pos, &s.a16, &s.bigram, &s.loop_step, &s.x0, &s.qabs, &s.olat, &s.ffa,
                     &s.rlogit, &s.moe_idx, &s.moe_w, &s.moe_pos, &s.moe_src, &s.moe_tile, &s.moe_h, &s.moe_a, &s.moe_y, &s.moe_a16, &s.zero_idx, &s.hin, &s.final_a, &s.loop_in, &s.cat,
-                    &s.h2, &s.h1_16, &s.h2_16, &s.f16, &s.den};
+                    &s.h2, &s.h1_16, &s.h2_16, &s.f16, &s.den, &s.embed_nw};
     for (DevBuf* b : bs) b->free();
     delete m->seq;
     m->seq = nullptr;
@@ -1704,6 +1748,8 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
     B2_CHECK_ARG(d.norm_kind == B2_NORM_RMS || (d.norm_kind == B2_NORM_DYT && par), "b2_seq_model_create: norm kind %d does not go with block form %d", d.norm_kind, d.block);
     B2_CHECK_ARG(!d.loop_mix || (par && d.loop_times >= 1), "b2_seq_model_create: the input mix belongs to a looped block of a parallel-block model");
     B2_CHECK_ARG(d.embed_scale == 0.f || d.bigram_buckets == 0, "b2_seq_model_create: a scaled embedding does not go with the hashed bigram rows");
+    B2_CHECK_ARG(!d.embed_norm || (d.bigram_buckets == 0 && !d.loop_mix && (d.loop_times <= 1 || d.loop_plain) && (d.embed_scale == 0.f || d.embed_scale == 1.f)),
+                 "b2_seq_model_create: a normed embedding does not go with bigram rows, a kept embedding output or a scale");
     B2_CHECK_ARG(d.input_conv_taps >= 0 && d.input_conv_taps <= 16, "b2_seq_model_create: 0..16 taps of the input convolution");
     B2_CHECK_ARG(d.input_conv_taps == 0 || d.block == B2_BLOCK_SANDWICH_RMS, "b2_seq_model_create: the input convolution belongs to the sandwich block");
     B2_CHECK_ARG(d.bigram_buckets >= 0 && d.logit_softcap >= 0.f, "b2_seq_model_create: negative bigram buckets or soft-cap");
@@ -1732,6 +1778,8 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
         SeqLayerInfo& L = s->layers[i];
         const b2_seq_layer_desc& l = L.d;
         const char* why = nullptr;
+        // (the linear scaling takes its factor alone)
+        const bool scaling_ok = !(l.rot_factor > 0.f) || l.rot_scaling == B2_ROT_LINEAR || (l.rot_original > 0.f && l.rot_fast > 0.f && l.rot_slow > 0.f && l.rot_base > 1.f);
         if (l.ff < 0) why = "negative feed-forward width";
         else if (l.type == B2_MIXER_MAMBA2) {
             if (l.m_heads < 1 || l.m_vdim < 1 || l.m_state < 1 || l.m_groups < 1 || l.m_heads % l.m_groups) why = "mamba2: heads must be a positive multiple of groups";
@@ -1757,7 +1805,7 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
             else if (l.la_rot_dim < 0 || l.la_q_rank < 0 || l.la_kv_from < 0) why = "latent attention: negative size";
             else if (l.la_rank < 1 || l.la_rank > 512 || l.la_rank + l.la_rot_dim > 768) why = "latent attention: latent size 1..512, with the rotated part at most 768";
             else if (l.la_rot_dim > 0 && (l.rot_dims < 1 || l.rot_dims > l.la_rot_dim || !(l.rot_base > 0.f))) why = "latent attention: rotated dimensions within the rotated part, positive base";
-            else if (l.rot_factor > 0.f && !(l.rot_original > 0.f && l.rot_fast > 0.f && l.rot_slow > 0.f && l.rot_base > 1.f)) why = "rotation: scaled frequencies need original, fast and slow";
+            else if (!scaling_ok) why = "rotation: scaled frequencies need original, fast and slow";
             else if (l.la_kv_from > 0) {
                 const int j = l.la_kv_from - 1;
                 if (j >= i) why = "latent attention: cache rows can only be read from an earlier layer";
@@ -1784,7 +1832,8 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
             else if (l.ga_sink == B2_SINK_HEAD && l.ga_maps == 2) why = "attention: two maps take no learned sinks";
             else if (l.ga_conv < 0 || l.ga_conv > 16) why = "attention: 0..16 convolution taps";
             else if (l.rot_dims < 0 || l.rot_dims > l.ga_dim || (l.rot_dims > 0 && !(l.rot_base > 0.f))) why = "attention: rotated dimensions within a head, positive base";
-            else if (l.rot_factor > 0.f && !(l.rot_original > 0.f && l.rot_fast > 0.f && l.rot_slow > 0.f && l.rot_base > 1.f)) why = "rotation: scaled frequencies need original, fast and slow";
+            else if (!scaling_ok) why = "rotation: scaled frequencies need original, fast and slow";
+            else if (l.ga_qkv_bias && l.ga_maps == 2) why = "attention: two maps take no projection biases";
             else if (l.ga_rot_values && !(l.rot_base > 0.f)) why = "attention: rotated values need a base";
             else if (l.mask_kind < B2_MASK_CAUSAL || l.mask_kind > B2_MASK_CHUNK || (l.mask_kind != B2_MASK_CAUSAL && l.mask_size < 1)) why = "mask: unknown kind or empty size";
             else if (l.mask_keep < 0 || (l.mask_keep > 0 && l.mask_kind != B2_MASK_WINDOW)) why = "mask: kept first positions belong to a window";
@@ -1828,16 +1877,16 @@ int b2_seq_model_create(const b2_seq_model_desc* desc, const b2_seq_layer_desc* 
         }
         const bool pre_mixer = l.type == B2_MIXER_LATENT_ATTN || l.type == B2_MIXER_HGRN2 || l.type == B2_MIXER_GQA_ATTN || l.type == B2_MIXER_GLA || l.type == B2_MIXER_MLSTM || l.type == B2_MIXER_DELTA;
         if (why == nullptr && (l.type == B2_MIXER_MLSTM || l.type == B2_MIXER_DELTA) && !par) why = "matrix memories need a parallel block";
-        if (why == nullptr && (l.rot_scaling < B2_ROT_YARN || l.rot_scaling > B2_ROT_BANDS)) why = "rotation: unknown scaling";
+        if (why == nullptr && (l.rot_scaling < B2_ROT_YARN || l.rot_scaling > B2_ROT_LINEAR)) why = "rotation: unknown scaling";
         if (why == nullptr && pre_mixer != (d.block != B2_BLOCK_POST_LN)) why = "this mixer does not go with the model's block form";
         if (why == nullptr && l.ff > 0) {
             if (l.ff_kind != B2_FF_RELU_SQ && d.block == B2_BLOCK_POST_LN) why = "this feed-forward needs a pre-norm or sandwich block";
             else if (l.ff_kind == B2_FF_MOE) {
-                if (l.moe_experts < 1 || l.moe_top < 1 || l.moe_top > 32 || l.moe_top > l.moe_experts) why = "moe: experts >= top >= 1, at most 32 choices";
-                else if (l.moe_groups < 1 || l.moe_experts % l.moe_groups || l.moe_keep < 1 || l.moe_keep > l.moe_groups) why = "moe: groups must divide experts, 1 <= keep <= groups";
+                if (l.moe_experts < 1 || l.moe_top < 1 || l.moe_top > 32 || l.moe_identity < 0 || l.moe_top > l.moe_experts + l.moe_identity) why = "moe: experts >= top >= 1, at most 32 choices";
+                else if (l.moe_groups < 1 || (l.moe_experts + l.moe_identity) % l.moe_groups || l.moe_keep < 1 || l.moe_keep > l.moe_groups) why = "moe: groups must divide experts, 1 <= keep <= groups";
                 else if (l.moe_shared_ff < 0) why = "moe: negative shared width";
-                else if (l.moe_score < 0 || l.moe_score > 1 || l.moe_group_score < 0 || l.moe_group_score > 1 || l.moe_act < 0 || l.moe_act > 1) why = "moe: unknown score, group score or activation";
-            } else if (l.ff_kind == B2_FF_CLAMP_GLU) {
+                else if (l.moe_score < 0 || l.moe_score > 1 || l.moe_group_score < 0 || l.moe_group_score > 1 || l.moe_act < 0 || l.moe_act > B2_MOE_ACT_CLAMP_GLU || l.ff_limit < 0.f) why = "moe: unknown score, group score or activation";
+            } else if (is_glu(l.ff_kind)) {
                 if (l.ff_limit < 0.f) why = "gated feed-forward: negative limit";
             } else if (l.ff_kind != B2_FF_RELU_SQ && l.ff_kind != B2_FF_POLYNORM && l.ff_kind != B2_FF_GELU) why = "unknown feed-forward kind";
         }

@@ -81,7 +81,8 @@ class SeqLayerDesc(_c.Structure):
                 ("ff_limit", _c.c_float), ("ff_act_slope", _c.c_float),
                 ("ga_key_values", _c.c_int32), ("rot_scaling", _c.c_int32),
                 ("ml_heads", _c.c_int32), ("ml_dim", _c.c_int32), ("ml_vdim", _c.c_int32), ("ml_cap", _c.c_float),
-                ("dn_heads", _c.c_int32), ("dn_kv_heads", _c.c_int32), ("dn_dim", _c.c_int32), ("dn_vdim", _c.c_int32), ("dn_conv", _c.c_int32)]
+                ("dn_heads", _c.c_int32), ("dn_kv_heads", _c.c_int32), ("dn_dim", _c.c_int32), ("dn_vdim", _c.c_int32), ("dn_conv", _c.c_int32),
+                ("ga_qkv_bias", _c.c_int32), ("moe_correction", _c.c_int32), ("moe_identity", _c.c_int32)]
 
 
 class SeqModelDesc(_c.Structure):
@@ -92,21 +93,21 @@ class SeqModelDesc(_c.Structure):
                 ("bigram_buckets", _c.c_int32), ("bigram_mul_prev", _c.c_int32), ("bigram_mul_cur", _c.c_int32),
                 ("loop_start", _c.c_int32), ("loop_stop", _c.c_int32), ("loop_times", _c.c_int32),
                 ("logit_scale", _c.c_float), ("input_conv_taps", _c.c_int32), ("embed_scale", _c.c_float), ("loop_plain", _c.c_int32),
-                ("norm_kind", _c.c_int32), ("tied_head", _c.c_int32), ("loop_mix", _c.c_int32)]
+                ("norm_kind", _c.c_int32), ("tied_head", _c.c_int32), ("loop_mix", _c.c_int32), ("embed_norm", _c.c_int32)]
 
 
 MIXER_MAMBA2, MIXER_PARALLEL, MIXER_LATENT_ATTN, MIXER_HGRN2, MIXER_GQA_ATTN, MIXER_GLA, MIXER_MLSTM, MIXER_DELTA = 1, 2, 3, 4, 5, 6, 7, 8
-FF_RELU_SQ, FF_POLYNORM, FF_MOE, FF_CLAMP_GLU, FF_GELU = 0, 1, 2, 3, 4
+FF_RELU_SQ, FF_POLYNORM, FF_MOE, FF_CLAMP_GLU, FF_GELU, FF_GELU_GLU = 0, 1, 2, 3, 4, 5
 BLOCK_POST_LN, BLOCK_PRE_RMS1, BLOCK_SANDWICH_RMS, BLOCK_PARALLEL_RMS, BLOCK_PARALLEL2 = 0, 1, 2, 3, 4
 NORM_RMS, NORM_DYT = 0, 1
 QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_ALL = 0, 1, 2
 SINK_NONE, SINK_FIXED, SINK_HEAD = 0, 1, 2
-ROT_YARN, ROT_BANDS = 0, 1
+ROT_YARN, ROT_BANDS, ROT_LINEAR = 0, 1, 2
 GATE_CHANNEL, GATE_HEAD, GATE_NONE = 0, 1, 2
 MASK_CAUSAL, MASK_WINDOW, MASK_CHUNK = 0, 1, 2
 MOE_SCORE_SIGMOID, MOE_SCORE_SOFTMAX = 0, 1
 MOE_GROUP_TOP2_SUM, MOE_GROUP_MAX = 0, 1
-MOE_ACT_SWIGLU, MOE_ACT_RELU_SQ = 0, 1
+MOE_ACT_SWIGLU, MOE_ACT_RELU_SQ, MOE_ACT_CLAMP_GLU = 0, 1, 2
 COMPUTE_BF16, COMPUTE_F32 = 0, 1
 
 

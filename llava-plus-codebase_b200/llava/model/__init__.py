@@ -14,16 +14,18 @@ MODEL_REGISTRY = {
     "Fezuzen": ("language_model.fezuzen", "FezuzenForCausalLM"),
     "Sofopel": ("language_model.sofopel", "SofopelForCausalLM"),
     "Ramosun": ("language_model.ramosun", "RamosunForCausalLM"),
+    "Kuvelix": ("language_model.kuvelix", "KuvelixForCausalLM"),
 }
 _LAZY = {"LlavaLlamaForCausalLM": "language_model.llava_llama", "LlavaConfig": "language_model.llava_llama",
          "KatadraForCausalLM": "language_model.katadra", "KatadraConfig": "language_model.katadra",
          "PefivikForCausalLM": "language_model.pefivik", "PefivikConfig": "language_model.pefivik",
          "FezuzenForCausalLM": "language_model.fezuzen", "FezuzenConfig": "language_model.fezuzen",
          "SofopelForCausalLM": "language_model.sofopel", "SofopelConfig": "language_model.sofopel",
-         "RamosunForCausalLM": "language_model.ramosun", "RamosunConfig": "language_model.ramosun"}
+         "RamosunForCausalLM": "language_model.ramosun", "RamosunConfig": "language_model.ramosun",
+         "KuvelixForCausalLM": "language_model.kuvelix", "KuvelixConfig": "language_model.kuvelix"}
 
 __all__ = ["LlavaConfig", "LlavaLlamaForCausalLM", "KatadraConfig", "KatadraForCausalLM", "PefivikConfig", "PefivikForCausalLM", "FezuzenConfig",
-           "FezuzenForCausalLM", "SofopelConfig", "SofopelForCausalLM", "RamosunConfig", "RamosunForCausalLM", "MODEL_REGISTRY",
+           "FezuzenForCausalLM", "SofopelConfig", "SofopelForCausalLM", "RamosunConfig", "RamosunForCausalLM", "KuvelixConfig", "KuvelixForCausalLM", "MODEL_REGISTRY",
            "model_class_for"]
 
 
