@@ -55,11 +55,11 @@ def parse_args():
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-configs", action="store_true", help="skip the side measurements of the other BASELINE configs")
-    ap.add_argument("--arch", default="llava", choices=["llava", "katadra", "pefivik", "fezuzen", "sofopel", "ramosun"],
+    ap.add_argument("--arch", default="llava", choices=["llava", "katadra", "pefivik", "fezuzen", "sofopel", "ramosun", "kuvelix"],
                     help="katadra: prefill / decode throughput of the layer-list decoder beside the LLaMA decoder of equal width, "
                          "depth and parameter count (random weights); the default workload and its JSON line are unchanged")
-    ap.add_argument("--widths", default="2048,4096", help="--arch katadra / pefivik / fezuzen / sofopel / ramosun: model widths to measure")
-    ap.add_argument("--ctx", type=int, default=2048, help="--arch katadra / pefivik / fezuzen / sofopel / ramosun: prompt length")
+    ap.add_argument("--widths", default="2048,4096", help="--arch katadra / pefivik / fezuzen / sofopel / ramosun / kuvelix: model widths to measure")
+    ap.add_argument("--ctx", type=int, default=2048, help="--arch katadra / pefivik / fezuzen / sofopel / ramosun / kuvelix: prompt length")
     return ap.parse_args()
 
 
@@ -1096,6 +1096,77 @@ def run_ramosun(args):
     print(json.dumps(out))
 
 
+def kuvelix_config(width):
+    """Four parallel-block layers of the sizes a model of this width would have: attention (heads of 128, four query heads per key/value
+    head, biases, head norms, 64 rotated entries slowed down by 4, a gate per channel) beside one dense gated GELU feed-forward of 11/8
+    width and three mixtures of 14 bounded gated experts of 3/8 width with 2 identity experts (4 choices among the best 2 of 4 groups),
+    about the parameters of Fezuzen's ungated mixtures with their shared expert."""
+    heads = width // 128
+    att = {"type": "attention", "mixer": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                          "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0}}}}
+    moe = {"kind": "moe", "expert": {"ff": 3 * width // 8, "limit": 7.0}, "router": {"experts": 14, "identity": 2, "groups": {"count": 4, "keep": 2}, "top": 4}}
+    return {"architecture": "Kuvelix", "width": width, "vocab": 32000, "norm": {"eps": 1e-6},
+            "layers": [dict(att, mlp={"kind": "dense", "ff": 11 * width // 8})] + [dict(att, mlp=moe)] * 3}
+
+
+def kuvelix_params(cfg):
+    """(matmul parameters a token multiplies with, function B -> parameters a decode step of B slots reads); a choice is an identity
+    expert as often as the identity experts' share of the router's rows says"""
+    W = cfg["width"]
+    fixed, per_expert, rows, experts, top = cfg["vocab"] * W, 0, 1, 1, 0
+    for layer in cfg["layers"]:
+        m, mlp = layer["mixer"], layer["mlp"]
+        H, G = m["heads"], m["kv_heads"]
+        fixed += (H * m["dim"] + G * m["dim"] + G * m["vdim"] + 2 * H * m["vdim"]) * W
+        if mlp["kind"] == "dense":
+            fixed += 3 * mlp["ff"] * W
+        else:
+            r = mlp["router"]
+            experts, top = r["experts"], r["top"]
+            rows = experts + r["identity"]
+            fixed += rows * W
+            per_expert += 3 * mlp["expert"]["ff"] * W
+    return int(fixed + top * experts / rows * per_expert), lambda B: fixed + per_expert * experts * (1.0 - (1.0 - top / rows) ** B)
+
+
+def run_kuvelix(args):
+    """Kuvelix beside Fezuzen, the package's closest model (grouped attention with a gate per channel, a mixture of experts behind a
+    group-limited softmax router in every layer, the same Linears), at equal width and depth."""
+    from oracle import fezuzen_oracle as FO
+    from oracle import kuvelix_oracle as VO
+    from llava.model import FezuzenConfig, FezuzenForCausalLM, KuvelixConfig, KuvelixForCausalLM
+    from llava._b2 import launch_count
+
+    dev = torch.device("cuda:0")
+    hbm, tfl, src = peaks()
+    pk = {"hbm_gbs": hbm, "bf16_tflops": tfl, "source": src}
+    S, N, layers = args.ctx, 64, 4
+    flush = torch.zeros(160 * 1024 * 1024 // 4, device=dev)  # 160 MB > 126 MB of L2
+    out = {"metric": "Kuvelix vs Fezuzen (layer-list decoders) at equal width and depth", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+           "peaks": pk, "prompt": S, "decode_steps": N, "l2": "160 MB written before every timed run", "sizes": []}
+    sampler = ClockSampler(0)
+    sampler.start()
+    launches0 = launch_count()
+    for width in [int(w) for w in args.widths.split(",")]:
+        row = {"width": width, "layers": layers}
+        for name, mk_cfg, mk_params, oracle, cfg_cls, model_cls in (
+                ("kuvelix", kuvelix_config, kuvelix_params, VO, KuvelixConfig, KuvelixForCausalLM),
+                ("fezuzen", lambda w_: fezuzen_config(w_, S), fezuzen_params, FO, FezuzenConfig, FezuzenForCausalLM)):
+            cfg = mk_cfg(width)
+            w = oracle.random_weights(cfg, seed=0)
+            params, params_read = mk_params(cfg)
+            model = model_cls(cfg_cls(**cfg), {k: torch.from_numpy(np.asarray(v, np.float32)).bfloat16() for k, v in w.items()}, device=dev, dtype=torch.bfloat16,
+                              max_batch=8, max_seq=S + N + 8, max_rows=S)
+            row[name + "_params_total"] = int(sum(v.size for k, v in w.items() if v.ndim == 2 and (k != "embed" or name == "kuvelix")))
+            del w
+            row[name] = measure_layer_list(model, args, S, N, flush, pk, params, params_read)
+            del model
+        out["sizes"].append(row)
+    out["clocks"] = sampler.stop()
+    out["gpu_launches"] = launch_count() - launches0
+    print(json.dumps(out))
+
+
 def run_katadra(args):
     from oracle import katadra_oracle as KO
     from llava.model import KatadraConfig, KatadraForCausalLM
@@ -1156,11 +1227,11 @@ def run_katadra(args):
 
 def main():
     args = parse_args()
-    if args.arch in ("katadra", "pefivik", "fezuzen", "sofopel", "ramosun"):
+    if args.arch in ("katadra", "pefivik", "fezuzen", "sofopel", "ramosun", "kuvelix"):
         if not torch.cuda.is_available():
             raise RuntimeError(f"bench.py --arch {args.arch} needs a B200")
         return {"katadra": run_katadra, "pefivik": run_pefivik, "fezuzen": run_fezuzen, "sofopel": run_sofopel,
-                "ramosun": run_ramosun}[args.arch](args)
+                "ramosun": run_ramosun, "kuvelix": run_kuvelix}[args.arch](args)
     if args.impl == "reference":
         run_reference(args)
     else:

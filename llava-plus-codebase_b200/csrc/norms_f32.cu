@@ -278,6 +278,55 @@ __global__ void embed_norm_kernel(const int32_t* __restrict__ tokens, const TT* 
     for (int c = threadIdx.x; c < cols; c += blockDim.x) x[r * cols + c] = (float)e[c] * mul * w[c];
 }
 
+// the same for rows of whole pieces of four entries, at most V per thread: one read of the row, weights loaded in front of the reduction
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(t.x << 16), __uint_as_float(t.x & 0xffff0000u), __uint_as_float(t.y << 16), __uint_as_float(t.y & 0xffff0000u));
+}
+template <typename TT, int V>
+__global__ void __launch_bounds__(256) embed_norm_reg_kernel(const int32_t* __restrict__ tokens, const TT* __restrict__ table, float* __restrict__ x,
+                                                             int cols, int vocab, int* err_flag, const float* __restrict__ w, float eps) {
+    __shared__ float red[33];
+    const size_t r = blockIdx.x;
+    const int t = tokens[r];
+    const bool ok = t >= 0 && t < vocab;
+    if (!ok && threadIdx.x == 0 && err_flag != nullptr) err_flag[0] = 1;
+    const TT* e = table + (size_t)(ok ? t : 0) * cols;
+    float4 v[V], g[V];
+    float q = 0.f;
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int c = (threadIdx.x + u * blockDim.x) * 4;
+        v[u] = g[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < cols) { v[u] = load4(e + c); g[u] = load4(w + c); }
+    }
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        q = fmaf(v[u].x, v[u].x, q); q = fmaf(v[u].y, v[u].y, q);
+        q = fmaf(v[u].z, v[u].z, q); q = fmaf(v[u].w, v[u].w, q);
+    }
+    const float norm = 1.f / sqrtf(block_sum(q, red) / (float)cols + eps), mul = ok ? norm : 0.f;
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+        const int c = (threadIdx.x + u * blockDim.x) * 4;
+        if (c < cols) *reinterpret_cast<float4*>(x + r * cols + c) = make_float4(v[u].x * mul * g[u].x, v[u].y * mul * g[u].y, v[u].z * mul * g[u].z, v[u].w * mul * g[u].w);
+    }
+}
+
+template <typename TT>
+int launch_embed_norm(const int32_t* tokens, const TT* table, float* x, int rows, int cols, int vocab, int* err_flag, const float* w, float eps, cudaStream_t st) {
+    const uintptr_t align = reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w);
+    if (cols % 4 == 0 && cols <= 8192 && (align & 15) == 0) {
+        if (cols <= 2048) embed_norm_reg_kernel<TT, 2><<<rows, 256, 0, st>>>(tokens, table, x, cols, vocab, err_flag, w, eps);
+        else embed_norm_reg_kernel<TT, 8><<<rows, 256, 0, st>>>(tokens, table, x, cols, vocab, err_flag, w, eps);
+    } else {
+        embed_norm_kernel<TT><<<rows, 256, 0, st>>>(tokens, table, x, cols, vocab, err_flag, w, eps);
+    }
+    B2_LAUNCH_CHECK();
+    return 0;
+}
+
 // post-norm add of one sublayer, pre-norm of the next, and (decode steps) the input convolution with its carried inputs
 __global__ void sandwich_norm_kernel(SandwichNormArgs a) {
     __shared__ float red[33];
@@ -600,13 +649,8 @@ int embed_rows_f32(const int32_t* tokens, const void* table, int table_dtype, fl
                    cudaStream_t st, float scale, const float* norm_w, float eps) {
     B2_CHECK_ARG(tokens && table && x && rows > 0 && (norm_w == nullptr || scale == 1.f), "embed_rows: bad argument");
     if (norm_w != nullptr) {
-        const int threads = cols >= 1024 ? 256 : 128;
-        if (table_dtype == DT_F32)
-            embed_norm_kernel<float><<<rows, threads, 0, st>>>(tokens, reinterpret_cast<const float*>(table), x, cols, vocab, err_flag, norm_w, eps);
-        else
-            embed_norm_kernel<__nv_bfloat16><<<rows, threads, 0, st>>>(tokens, reinterpret_cast<const __nv_bfloat16*>(table), x, cols, vocab, err_flag, norm_w, eps);
-        B2_LAUNCH_CHECK();
-        return 0;
+        if (table_dtype == DT_F32) return launch_embed_norm(tokens, reinterpret_cast<const float*>(table), x, rows, cols, vocab, err_flag, norm_w, eps, st);
+        return launch_embed_norm(tokens, reinterpret_cast<const __nv_bfloat16*>(table), x, rows, cols, vocab, err_flag, norm_w, eps, st);
     }
     if (table_dtype == DT_F32)
         embed_rows_kernel<float><<<rows, 128, 0, st>>>(tokens, reinterpret_cast<const float*>(table), x, cols, vocab, err_flag, scale);
